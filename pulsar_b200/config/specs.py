@@ -18,6 +18,7 @@ class NormSpec:
     eps: float
     suffix: str = "weight"   # the weight's tensor name is the part's prefix + this ("" where the prefix is the whole name)
     scalar: bool = False     # the weight is a single number (a tensor without dimensions) for all coordinates
+    about_one: bool = False  # the tensor holds the weight's distance from one: the norm multiplies by 1 + w
 
 
 @dataclass(frozen=True)
@@ -71,6 +72,13 @@ class MixerSpec:
     differential: Optional[float] = None
     norm_eps: float = 0.0            # eps of norms inside the mixer (the differential form's norm of a head's output)
     q_temperature: Optional[Tuple[float, int]] = None   # (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
+    qk_norm_whole: bool = False      # with qk_norm_eps: one weighted RMS norm over all query heads' elements together (and one over the key heads'), before the rotation
+    rotate_neighbours: bool = False  # the rotation pairs elements 2i and 2i + 1 of a head (else i and i + rotary_dim / 2)
+    # The value of a position is turned by it over these dimensions (pairs of neighbours) and cached so; every head's output
+    # is turned back by the query's position.  None: values as projected.
+    value_position: Optional[PositionSpec] = None
+    sigmoid_weights: bool = False    # no softmax: a visible key's weight is sigmoid(score), not normalised over the keys
+    score_bias: bool = False         # with sigmoid_weights: a learned number per head joins the score (tensor role "score_bias")
     extra: Tuple[Tuple[str, object], ...] = ()   # free-form parameters of other kinds
 
     def option(self, name, default=None):

@@ -11,7 +11,12 @@
 //     floor(p / chunk) * chunk (chunk > 0; chunks are counted from position 0 of the sequence);
 //     with keep_first > 0 the keys 0 .. keep_first - 1 stay visible below lo as well (at their true positions);
 //   * with softcap > 0 the scaled score becomes softcap * tanh(score / softcap) (before the distance bias);
-//   * with `sinks` [Hq] the softmax's denominator holds one more term per head, exp(sinks[h]), that has no value.
+//   * with `sinks` [Hq] the softmax's denominator holds one more term per head, exp(sinks[h]), that has no value;
+//   * with `sigmoid` there is no softmax: a visible key's weight is 1 / (1 + exp(-(score + score_bias[h]))) (score_bias
+//     optional), and the weights are not normalised over the keys;
+//   * with `out_cos` / `out_sin` [N, Dv / 2] the finished output row of a token turns back by the token's angles: columns
+//     2m and 2m + 1 are a pair (u, v) -> (u cos + v sin, v cos - u sin), before the one rounding (values that were cached
+//     turned by their own positions then enter by the difference of the two).
 // Queries come in float32 (rotation and score are 32-bit arithmetic whatever the cache holds);
 // scores, the running maximum, the sums and the output accumulate in float32 with expf.
 //
@@ -59,7 +64,16 @@ struct GeneralShape {
     float softcap;      // > 0: scaled scores are capped to softcap * tanh(score / softcap)
     int v_share;        // consecutive key heads that read one value head (the value pool has Hkv / v_share heads); 1: a value head per key head
     int out_f32;        // the output rows are float32 whatever the pools' type (what follows subtracts them from one another)
+    int sigmoid;        // a key's weight is the sigmoid of its score (+ score_bias[head]) and nothing is normalised
+    const float *score_bias, *out_cos, *out_sin;
 };
+
+__device__ __forceinline__ float sigmoid_weight(float s) { return 1.0f / (1.0f + expf(-s)); }
+
+// Columns 2m and 2m + 1 of a finished row turn back by angle m of the row's token; `even`: this is the pair's first column.
+__device__ __forceinline__ float turned_back(float own, float other, int m, int even, const float* cos_row, const float* sin_row) {
+    return even ? own * cos_row[m] + other * sin_row[m] : own * cos_row[m] - other * sin_row[m];
+}
 
 template <typename T>
 __device__ __forceinline__ void store_out(T* out, size_t at, float v, int out_f32) {
@@ -107,6 +121,7 @@ paged_attention_general_kernel(const float* __restrict__ q, const T* __restrict_
     for (int i = threadIdx.x; i < Dk; i += blockDim.x) q_s[i] = qv[i] * sh.scale;
     __syncthreads();
 
+    const float bias = (sh.sigmoid && sh.score_bias) ? sh.score_bias[h] : 0.0f;
     float m_run = -INFINITY, l_run = 0.0f;
     float acc[ACC];
 #pragma unroll
@@ -135,13 +150,18 @@ paged_attention_general_kernel(const float* __restrict__ q, const T* __restrict_
             for (; d < Dk; ++d) dot = fmaf(q_s[d], to_float(kr[d]), dot);
             sc = cap_score(dot, sh.softcap) - slope * (float)(p - j);
         }
-        const float m_new = fmaxf(m_run, warp_max(sc));      // finite: every tile in range has a visible key
-        const float pv = valid ? expf(sc - m_new) : 0.0f;
-        const float corr = expf(m_run - m_new);               // 0 on the first tile (m_run = -inf)
-        l_run = l_run * corr + warp_sum(pv);
-        m_run = m_new;
+        float pv;
+        if (sh.sigmoid) {                                     // uniform over the grid
+            pv = valid ? sigmoid_weight(sc + bias) : 0.0f;
+        } else {
+            const float m_new = fmaxf(m_run, warp_max(sc));   // finite: every tile in range has a visible key
+            pv = valid ? expf(sc - m_new) : 0.0f;
+            const float corr = expf(m_run - m_new);           // 0 on the first tile (m_run = -inf)
+            l_run = l_run * corr + warp_sum(pv);
+            m_run = m_new;
 #pragma unroll
-        for (int i = 0; i < ACC; ++i) acc[i] *= corr;
+            for (int i = 0; i < ACC; ++i) acc[i] *= corr;
+        }
         __syncwarp();
         p_s[warp * 32 + lane] = pv;
         __syncwarp();
@@ -177,12 +197,25 @@ paged_attention_general_kernel(const float* __restrict__ q, const T* __restrict_
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) { f[w] = (m_s[w] == -INFINITY) ? 0.0f : expf(m_s[w] - m_all); l_all += l_s[w] * f[w]; }
     if (sinks) l_all += expf(sinks[h] - m_all);
+    if (sh.sigmoid) {                                         // the warps' sums add up as they are
+        l_all = 1.0f;
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) f[w] = 1.0f;
+    }
     const size_t ov = ((size_t)t * sh.Hq + h) * Dv;
-    for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
+    auto column = [&](int d) {
         float o = 0.0f;
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) o += acc_s[w * Dv + d] * f[w];
-        store_out(out, ov + d, o / l_all, sh.out_f32);
+        return o / l_all;
+    };
+    for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
+        float o = column(d);
+        if (sh.out_cos) {
+            const size_t at = (size_t)t * (Dv >> 1);
+            o = turned_back(o, column(d ^ 1), d >> 1, !(d & 1), sh.out_cos + at, sh.out_sin + at);
+        }
+        store_out(out, ov + d, o, sh.out_f32);
     }
 }
 
@@ -282,7 +315,7 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
 
     // this thread's four rows
     int pos[4], lo_r[4], tok[4], head[4];
-    float slope[4];
+    float slope[4], bias[4];
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
         const int row = warp * 4 + r;
@@ -296,6 +329,7 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
         if (sh.chunk > 0 && pos[r] >= 0 && (pos[r] / sh.chunk) * sh.chunk > lo) lo = (pos[r] / sh.chunk) * sh.chunk;
         lo_r[r] = lo;
         slope[r] = slopes ? slopes[head[r]] : 0.0f;
+        bias[r] = (sh.sigmoid && sh.score_bias) ? sh.score_bias[head[r]] : 0.0f;
     }
     // the rows' queries, 16 bytes at a time, all copies in flight at once (the scale enters with the scores)
     {
@@ -376,6 +410,10 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
             const float v = vis ? (sh.softcap > 0.0f ? cap_score(sc[r] * sh.scale, sh.softcap) - slope[r] * (float)(pos[r] - j)
                                                      : fmaf(sc[r], sh.scale, -slope[r] * (float)(pos[r] - j)))
                                 : -INFINITY;
+            if (sh.sigmoid) {                               // uniform over the grid
+                p_s[(warp * 4 + r) * kTile + lane] = vis ? sigmoid_weight(v + bias[r]) : 0.0f;
+                continue;
+            }
             const float m_new = fmaxf(m_run[r], warp_max(v));
             float pv = 0.0f, corr = 1.0f;
             if (m_new != -INFINITY) {                       // uniform over the warp
@@ -422,11 +460,17 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
         if (warp * 4 + r >= n_rows) continue;
         const size_t row = (size_t)tok[r] * sh.Hq + head[r];
         if (ts.n_splits == 1) {
-            const float inv = 1.0f / (sinks ? l_run[r] + expf(sinks[head[r]] - m_run[r]) : l_run[r]);
+            const float inv = sh.sigmoid ? 1.0f : 1.0f / (sinks ? l_run[r] + expf(sinks[head[r]] - m_run[r]) : l_run[r]);
+            const size_t at = (size_t)tok[r] * (Dv >> 1);
 #pragma unroll
             for (int i = 0; i < ACC; ++i) {
                 const int c = lane + 32 * i;
-                if (c < Dv) store_out(out, row * Dv + c, acc[r][i] * inv, sh.out_f32);
+                float o = acc[r][i] * inv;
+                if (sh.out_cos) {                           // uniform over the grid; the pair's other column is the neighbouring lane's
+                    const float other = __shfl_xor_sync(0xffffffffu, o, 1);
+                    if (c < Dv) o = turned_back(o, other, c >> 1, !(c & 1), sh.out_cos + at, sh.out_sin + at);
+                }
+                if (c < Dv) store_out(out, row * Dv + c, o, sh.out_f32);
             }
         } else {
             float* pp = partial + (row * ts.n_splits + split) * (Dv + 2);
@@ -442,11 +486,31 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
 
 // out[row] = sum over the splits, in their order, of their partial outputs weighted by exp(m_split - m_all), over the
 // weighted sum of their sums.  One block per (token, head).
+// (With `sigmoid` the partial outputs are added as they are; a row's columns turn back where the launch says so.)
 template <typename T>
 __global__ void general_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, const float* __restrict__ sinks,
-                                       int Hq, int n_splits, int Dv, int out_f32) {
+                                       int n_splits, const GeneralShape sh) {
     const size_t row = blockIdx.x;
+    const int Hq = sh.Hq, Dv = sh.Dv, out_f32 = sh.out_f32;
     const float* pp = partial + row * n_splits * (Dv + 2);
+    if (sh.sigmoid) {                                        // uniform over the grid
+        auto column = [&](int c) {
+            float o = 0.0f;
+            for (int z = 0; z < n_splits; ++z) o += pp[(size_t)z * (Dv + 2) + 2 + c];
+            return o;
+        };
+        if (sh.out_cos) {                                    // a thread takes both columns of a pair
+            const size_t at = row / Hq * (Dv >> 1);
+            for (int m = threadIdx.x; m < (Dv >> 1); m += blockDim.x) {
+                const float u = column(2 * m), v = column(2 * m + 1);
+                store_out(out, row * Dv + 2 * m, turned_back(u, v, m, 1, sh.out_cos + at, sh.out_sin + at), out_f32);
+                store_out(out, row * Dv + 2 * m + 1, turned_back(v, u, m, 0, sh.out_cos + at, sh.out_sin + at), out_f32);
+            }
+        } else {
+            for (int c = threadIdx.x; c < Dv; c += blockDim.x) store_out(out, row * Dv + c, column(c), out_f32);
+        }
+        return;
+    }
     float m_all = -INFINITY;
     for (int z = 0; z < n_splits; ++z) m_all = fmaxf(m_all, pp[(size_t)z * (Dv + 2)]);
     float l_all = 0.0f;
@@ -455,13 +519,21 @@ __global__ void general_combine_kernel(const float* __restrict__ partial, T* __r
         if (m != -INFINITY) l_all += pp[(size_t)z * (Dv + 2) + 1] * expf(m - m_all);
     }
     if (sinks) l_all += expf(sinks[row % Hq] - m_all);
-    for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
+    auto column = [&](int c) {
         float o = 0.0f;
         for (int z = 0; z < n_splits; ++z) {
             const float m = pp[(size_t)z * (Dv + 2)];
             if (m != -INFINITY) o += pp[(size_t)z * (Dv + 2) + 2 + c] * expf(m - m_all);
         }
-        store_out(out, row * Dv + c, o / l_all, out_f32);
+        return o / l_all;
+    };
+    for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
+        float o = column(c);
+        if (sh.out_cos) {
+            const size_t at = row / Hq * (Dv >> 1);
+            o = turned_back(o, column(c ^ 1), c >> 1, !(c & 1), sh.out_cos + at, sh.out_sin + at);
+        }
+        store_out(out, row * Dv + c, o, out_f32);
     }
 }
 
@@ -488,7 +560,7 @@ int launch_tiled(const float* q, const void* k_pool, const void* v_pool, void* o
     if (status == 0 && ts.n_splits > 1) {
         int b = 32;
         while (b < ts.g.Dv && b < 256) b <<= 1;
-        general_combine_kernel<T><<<n_tokens * ts.g.Hq, b, 0, stream>>>(partial, (T*)out, sinks, ts.g.Hq, ts.n_splits, ts.g.Dv, ts.g.out_f32);
+        general_combine_kernel<T><<<n_tokens * ts.g.Hq, b, 0, stream>>>(partial, (T*)out, sinks, ts.n_splits, ts.g);
         status = launch_status();
     }
     return status;
@@ -553,20 +625,28 @@ __global__ void qkv_split_write_kernel(const T* __restrict__ qkv, float* __restr
     for (int i = lane; i < D; i += 32) dst[i] = src[i];
 }
 
+// Sigmoid weights have no denominator that a sink could join; turning back pairs the columns of a row.
+bool weighting_ok(int sigmoid, const float* score_bias, const float* sinks, const float* out_cos, const float* out_sin, int Dv) {
+    return !(sigmoid && sinks) && !(score_bias && !sigmoid) && ((out_cos == nullptr) == (out_sin == nullptr)) && !(out_cos && Dv % 2);
+}
+
 }  // namespace
 
+// sigmoid, score_bias (float32 [Hq] or null), out_cos / out_sin (float32 [n_tokens, Dv / 2] or null): see the head of this file.
 PB_EXPORT int pb_paged_attention_general(int dtype, const float* q, const void* k_pool, const void* v_pool, void* out,
                                          const int* block_table, int table_stride, const int* cu_q, const int* kv_len,
                                          const int* seq_of_token, const float* slopes, int n_tokens, int Hq, int Hkv, int Dk,
                                          int Dv, int k_stride, int v_stride, int page_size, float scale, int window, int chunk,
-                                         int keep_first, float softcap, const float* sinks, int v_share, int out_f32, cudaStream_t stream) {
+                                         int keep_first, float softcap, const float* sinks, int v_share, int out_f32, int sigmoid,
+                                         const float* score_bias, const float* out_cos, const float* out_sin, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (!weighting_ok(sigmoid, score_bias, sinks, out_cos, out_sin, Dv)) return PB_ERR_BAD_SIZE;
     if (Dk <= 0 || Dv <= 0 || Dk > 4096 || Dv > 1024 || Hkv <= 0 || Hq <= 0 || Hq % Hkv || page_size <= 0 || k_stride < Dk ||
         v_stride < Dv || window < 0 || chunk < 0 || keep_first < 0 || !(softcap >= 0.0f) || v_share <= 0 || Hkv % v_share)
         return PB_ERR_BAD_SIZE;
     if (Hq > 65535) return PB_ERR_TOO_LARGE;
     GeneralShape sh{Hq, Hkv, Dk, Dv, k_stride, v_stride, page_size, window, chunk, table_stride, 0, scale, keep_first, softcap, v_share,
-                    out_f32 != 0};
+                    out_f32 != 0, sigmoid != 0, score_bias, out_cos, out_sin};
     if (dtype == PB_F32)
         return dispatch_general<float>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, seq_of_token, slopes, sinks, n_tokens, sh,
                                        stream);
@@ -612,8 +692,10 @@ PB_EXPORT int pb_paged_attention_general_tiled(int dtype, const float* q, const 
                                                const int* kv_len, const float* slopes, int n_tokens, int n_seqs, int row_tiles,
                                                int n_splits, int Hq, int Hkv, int Dk, int Dv, int k_stride, int v_stride,
                                                int page_size, float scale, int window, int chunk, int keep_first, float softcap,
-                                               const float* sinks, int v_share, int out_f32, cudaStream_t stream) {
+                                               const float* sinks, int v_share, int out_f32, int sigmoid, const float* score_bias,
+                                               const float* out_cos, const float* out_sin, cudaStream_t stream) {
     if (n_tokens <= 0 || row_tiles <= 0) return 0;
+    if (!weighting_ok(sigmoid, score_bias, sinks, out_cos, out_sin, Dv)) return PB_ERR_BAD_SIZE;
     if (v_share <= 0 || Hkv % v_share) return PB_ERR_BAD_SIZE;
     if (!pb_attention_general_tiled_supported(dtype, k_pool, v_pool, Hq, Hkv, Dk, Dv, k_stride, v_stride)) return PB_ERR_BAD_SIZE;
     if (page_size <= 0 || window < 0 || chunk < 0 || keep_first < 0 || !(softcap >= 0.0f) || n_splits < 1 || n_splits > 65535 ||
@@ -622,7 +704,7 @@ PB_EXPORT int pb_paged_attention_general_tiled(int dtype, const float* q, const 
     if (Hkv > 65535) return PB_ERR_TOO_LARGE;
     TiledShape ts{};
     ts.g = GeneralShape{Hq, Hkv, Dk, Dv, k_stride, v_stride, page_size, window, chunk, table_stride, 0, scale, keep_first, softcap, v_share,
-                        out_f32 != 0};
+                        out_f32 != 0, sigmoid != 0, score_bias, out_cos, out_sin};
     ts.n_seqs = n_seqs;
     ts.n_splits = n_splits;
     if (dtype == PB_F32) {

@@ -14,7 +14,11 @@
 // absolute key indices and taken in ascending order; a tile in which a row sees nothing leaves the row as it was.
 // Kept first keys (keep_first > 0: keys 0 .. keep_first - 1 stay visible below the window), a cap on the scaled score
 // (softcap > 0: softcap * tanh(score / softcap) in float32, through ex2.approx like the softmax's exponentials) and a
-// sink per head (one more term exp(sinks[h]) in the softmax's denominator) as in the CUDA-core kernels.
+// sink per head (one more term exp(sinks[h]) in the softmax's denominator) as in the CUDA-core kernels.  With sigmoid weights
+// (kSigmoid: weight 1 / (1 + exp(-(score + score_bias[h]))), nothing normalised) there is no maximum, no rescaling and no sum;
+// the exponential comes from ex2.approx and the reciprocal from an approximate division (relative error 2^-21 of the weight).
+// Output rows may turn back by their token's angles before they are rounded (out_cos / out_sin, pairs of neighbours: a lane
+// holds both columns of a pair).
 #include "mma_common.cuh"
 
 namespace {
@@ -52,6 +56,7 @@ struct TcShape {
     float softcap;
     int v_share;        // consecutive key heads that read one value head (the value pool has Hkv / v_share heads)
     int out_f32;        // the output rows are float32: the accumulators go out as they are, without the round to bfloat16
+    const float *score_bias, *out_cos, *out_sin;
 };
 
 __device__ __forceinline__ int lowest_key(int pos, const TcShape& sh) {
@@ -61,7 +66,7 @@ __device__ __forceinline__ int lowest_key(int pos, const TcShape& sh) {
     return lo;
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool kSigmoid>
 __global__ void __launch_bounds__(kWarps * 32, 2)
 general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                   bf16* __restrict__ out, const int* __restrict__ block_table, const int* __restrict__ cu_q,
@@ -146,6 +151,7 @@ general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, 
     const float sl2 = sh.scale * kLog2e;
     const float cap_in = sh.softcap > 0.0f ? sh.scale / sh.softcap : 0.0f;
     const float slope2 = slopes ? slopes[head] * kLog2e : 0.0f;
+    const float bias2 = (kSigmoid && sh.score_bias) ? sh.score_bias[head] * kLog2e : 0.0f;
     const int r0 = min(warp * 16 + g, rows - 1), r1 = min(warp * 16 + g + 8, rows - 1);
     const int pos0 = pos_first + r0, pos1 = pos_first + r1;
     const int lo0 = lowest_key(pos0, sh), lo1 = lowest_key(pos1, sh);
@@ -208,12 +214,16 @@ general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, 
                         else
                             v = fmaf(sc[n][e], sl2, -slope2 * (float)(pos - key));
                     }
+                    if (kSigmoid) {                         // the weight itself
+                        sc[n][e] = vis ? __fdividef(1.0f, 1.0f + ex2(-(v + bias2))) : 0.0f;
+                        continue;
+                    }
                     sc[n][e] = v;
                     tmax[e >> 1] = fmaxf(tmax[e >> 1], v);
                 }
-            float corr[2], m_safe[2];
+            float corr[2] = {1.0f, 1.0f}, m_safe[2] = {0.0f, 0.0f};
 #pragma unroll
-            for (int r = 0; r < 2; ++r) {
+            for (int r = 0; r < (kSigmoid ? 0 : 2); ++r) {
                 float mx = tmax[r];
                 mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
                 mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -223,7 +233,7 @@ general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, 
                 m_run[r] = m_new;
                 l_run[r] *= corr[r];
             }
-            if (__any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f)) {
+            if (!kSigmoid && __any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f)) {
 #pragma unroll
                 for (int i = 0; i < kNTiles; ++i) {
                     o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1];
@@ -237,6 +247,10 @@ general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, 
                 for (int n = 0; n < 2; ++n)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
+                        if (kSigmoid) {
+                            pv[n][e] = sc[2 * kk + n][e];
+                            continue;
+                        }
                         pv[n][e] = ex2(sc[2 * kk + n][e] - m_safe[e >> 1]);
                         l_run[e >> 1] += pv[n][e];
                     }
@@ -272,7 +286,21 @@ general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, 
         l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
         if (sinks != nullptr && m_run[r] != -INFINITY) l_run[r] += ex2(fmaf(sinks[head], kLog2e, -m_run[r]));
     }
-    const float inv0 = l_run[0] > 0.0f ? 1.0f / l_run[0] : 0.0f, inv1 = l_run[1] > 0.0f ? 1.0f / l_run[1] : 0.0f;
+    const float inv0 = kSigmoid ? 1.0f : l_run[0] > 0.0f ? 1.0f / l_run[0] : 0.0f;
+    const float inv1 = kSigmoid ? 1.0f : l_run[1] > 0.0f ? 1.0f / l_run[1] : 0.0f;
+    if (sh.out_cos != nullptr) {                             // columns 8 i + 2 t and the next are pair 4 i + t of rows r0 and r1
+        const size_t at0 = (size_t)(q0 + m0 + r0) * (DV / 2), at1 = (size_t)(q0 + m0 + r1) * (DV / 2);
+#pragma unroll
+        for (int i = 0; i < kNTiles; ++i) {
+            const float c0 = sh.out_cos[at0 + 4 * i + t], s0 = sh.out_sin[at0 + 4 * i + t];
+            const float c1 = sh.out_cos[at1 + 4 * i + t], s1 = sh.out_sin[at1 + 4 * i + t];
+            const float u0 = o[i][0], u1 = o[i][2];
+            o[i][0] = u0 * c0 + o[i][1] * s0;
+            o[i][1] = o[i][1] * c0 - u0 * s0;
+            o[i][2] = u1 * c1 + o[i][3] * s1;
+            o[i][3] = o[i][3] * c1 - u1 * s1;
+        }
+    }
     if (sh.out_f32) {
         // a lane's accumulators are pairs of neighbours in rows g and g + 8 of the warp's 16: 8 bytes a store, 32 in a row per quad
         float* out32 = reinterpret_cast<float*>(out);
@@ -309,7 +337,7 @@ general_tc_kernel(const float* __restrict__ q, const bf16* __restrict__ k_pool, 
     }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool kSigmoid>
 int launch_general_tc(const float* q, const void* k_pool, const void* v_pool, void* out, const int* block_table, const int* cu_q,
                       const int* kv_len, const float* slopes, const float* sinks, int n_q_tiles, const TcShape& sh,
                       cudaStream_t stream) {
@@ -317,12 +345,12 @@ int launch_general_tc(const float* q, const void* k_pool, const void* v_pool, vo
     constexpr int smem = 2 * kBM * DK * 2 + 2 * kBN * (DK + DV) * 2;
     static bool configured = false;
     if (!configured) {
-        const cudaError_t rc = cudaFuncSetAttribute(general_tc_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        const cudaError_t rc = cudaFuncSetAttribute(general_tc_kernel<DK, DV, kSigmoid>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (rc != cudaSuccess) return (int)rc;
         configured = true;
     }
     dim3 grid(n_q_tiles, sh.Hq);
-    general_tc_kernel<DK, DV><<<grid, kWarps * 32, smem, stream>>>(q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, block_table,
+    general_tc_kernel<DK, DV, kSigmoid><<<grid, kWarps * 32, smem, stream>>>(q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, block_table,
                                                                    cu_q, kv_len, slopes, sinks, sh, pool_bounds_now());
     return launch_status();
 }
@@ -346,19 +374,22 @@ PB_EXPORT int pb_paged_attention_general_tc(int dtype, const float* q, const voi
                                             const int* block_table, int table_stride, const int* cu_q, const int* kv_len,
                                             const float* slopes, int n_seqs, int n_q_tiles, int Hq, int Hkv, int Dk, int Dv,
                                             int k_stride, int v_stride, int page_size, float scale, int window, int chunk,
-                                            int keep_first, float softcap, const float* sinks, int v_share, int out_f32, cudaStream_t stream) {
+                                            int keep_first, float softcap, const float* sinks, int v_share, int out_f32, int sigmoid,
+                                            const float* score_bias, const float* out_cos, const float* out_sin, cudaStream_t stream) {
     if (n_seqs <= 0 || n_q_tiles <= 0) return 0;
+    if ((sigmoid && sinks) || (score_bias && !sigmoid) || (out_cos == nullptr) != (out_sin == nullptr)) return PB_ERR_BAD_SIZE;
     if (v_share <= 0 || Hkv % v_share) return PB_ERR_BAD_SIZE;
     if (!pb_attention_general_tc_supported(dtype, q, k_pool, v_pool, Hq, Hkv, Dk, Dv, k_stride, v_stride) || ((uintptr_t)out % 16))
         return PB_ERR_BAD_SIZE;
     if (page_size <= 0 || window < 0 || chunk < 0 || keep_first < 0 || !(softcap >= 0.0f)) return PB_ERR_BAD_SIZE;
     const TcShape sh{n_seqs, Hq, Hkv, k_stride, v_stride, page_size, window, chunk, table_stride, scale, keep_first, softcap, v_share,
-                     out_f32 != 0};
-    if (Dk == 64 && Dv == 128)
-        return launch_general_tc<64, 128>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, slopes, sinks, n_q_tiles, sh, stream);
-    if (Dk == 64)
-        return launch_general_tc<64, 64>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, slopes, sinks, n_q_tiles, sh, stream);
-    if (Dk == 128)
-        return launch_general_tc<128, 128>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, slopes, sinks, n_q_tiles, sh, stream);
-    return launch_general_tc<192, 128>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, slopes, sinks, n_q_tiles, sh, stream);
+                     out_f32 != 0, score_bias, out_cos, out_sin};
+#define PB_TC(DK, DV)                                                                                                             \
+    return sigmoid ? launch_general_tc<DK, DV, true>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, slopes, sinks, n_q_tiles, sh, stream) \
+                   : launch_general_tc<DK, DV, false>(q, k_pool, v_pool, out, block_table, cu_q, kv_len, slopes, sinks, n_q_tiles, sh, stream)
+    if (Dk == 64 && Dv == 128) PB_TC(64, 128);
+    if (Dk == 64) PB_TC(64, 64);
+    if (Dk == 128) PB_TC(128, 128);
+    PB_TC(192, 128);
+#undef PB_TC
 }

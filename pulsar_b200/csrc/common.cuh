@@ -107,6 +107,12 @@ __device__ __forceinline__ float gated(float g, float u, const GatedInter& p) {
     return g / (1.0f + expf(-p.alpha * g)) * (u + p.shift);
 }
 
+// max(x, 0)^2: the activation of ungated feed-forwards that the products' epilogues can apply.
+__device__ __forceinline__ float squared_relu(float x) {
+    const float r = fmaxf(x, 0.0f);
+    return r * r;
+}
+
 // Programmatic dependent launch.  A kernel launched through launch_pdl may be brought onto the
 // SMs while the kernel before it on the stream is finishing: as soon as every block of that
 // kernel has called pdl_trigger (or exited).  It must call pdl_wait before it touches anything

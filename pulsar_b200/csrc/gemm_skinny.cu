@@ -16,7 +16,7 @@
 //
 // Epilogues: plain (bfloat16 or float32 output), or SwiGLU: the block's 16 rows are 8 gate
 // rows and the 8 up rows that belong to them, and it writes silu(gate) * up (float32
-// gating, one rounding), so the [M, 2I] intermediate never exists.
+// gating, one rounding), so the [M, 2I] intermediate never exists; or the squared ReLU max(., 0)^2 of the plain product.
 //
 // The reference calls at::linear three times for q/k/v, once for o, twice for gate/up and
 // once for down, plus two elementwise kernels for the gating
@@ -40,7 +40,10 @@ __device__ __forceinline__ uint4 load_stream(const void* p) {      // weights: r
     return v;
 }
 
-enum { kPlain = 0, kSwiGLU = 1 };
+enum { kPlain = 0, kSwiGLU = 1, kSquaredReLU = 2 };      // kSquaredReLU: the plain product's shape, max(., 0)^2 on the way out
+
+template <int MODE>
+__device__ __forceinline__ float activated(float v) { return MODE == kSquaredReLU ? squared_relu(v) : v; }
 
 // NT: n-tiles of 8 tokens.  Mode kSwiGLU: rows r of the block are gate rows 8*b + r (r < 8) and up rows
 // inter + 8*b + (r - 8); the output has `inter` columns.
@@ -142,7 +145,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, OutT*
             float acc = 0.0f;
 #pragma unroll
             for (int wi = 0; wi < kWarps; ++wi) acc += red[wi][r][token];
-            out[(size_t)token * N + blockIdx.x * kRows + r] = from_float<OutT>(acc);
+            out[(size_t)token * N + blockIdx.x * kRows + r] = from_float<OutT>(activated<MODE>(acc));
         }
     }
 }
@@ -430,7 +433,7 @@ skinny_wide_body(const bf16* __restrict__ x, const bf16* __restrict__ w, OutT* _
                     square_s[token][r] = x_new * x_new;
                 }
             } else {
-                *dst = from_float<OutT>(acc);
+                *dst = from_float<OutT>(activated<MODE>(acc));
             }
         }
         if constexpr (kAcc) {
@@ -593,7 +596,7 @@ gemm_skinny_tall_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, 
             float acc = 0.0f;
 #pragma unroll
             for (int wi = 0; wi < kWarps; ++wi) acc += red[wi][r][token];
-            out[(size_t)token * N + blockIdx.x * (kTallGroups * kRows) + r] = from_float<OutT>(acc);
+            out[(size_t)token * N + blockIdx.x * (kTallGroups * kRows) + r] = from_float<OutT>(activated<MODE>(acc));
         }
     }
 }
@@ -633,6 +636,10 @@ int launch_wide(int mode, int out_dtype, const bf16* xp, const bf16* wp, void* o
         if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
         return launch_pdl(gemm_skinny_wide_kernel<NT, kSwiGLU, bf16, kU, kEvictFirst>, inter / 8, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, inter);
     }
+    if (mode == kSquaredReLU) {
+        if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+        return launch_pdl(gemm_skinny_wide_kernel<NT, kSquaredReLU, bf16, kU, kEvictFirst>, N / kRows, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
+    }
     if (out_dtype == PB_BF16)
         return launch_pdl(gemm_skinny_wide_kernel<NT, kPlain, bf16, kU, kEvictFirst>, N / kRows, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
     return launch_pdl(gemm_skinny_wide_kernel<NT, kPlain, float, kU, kEvictFirst>, N / kRows, kWarps * 32, 0, stream, xp, wp, (float*)out, M, N, K, 0);
@@ -644,6 +651,10 @@ int launch_prefetch(int mode, int out_dtype, const bf16* xp, const bf16* wp, voi
         const GatedInter inter = gating_now(N / 2);
         if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
         return launch_pdl(gemm_skinny_wide_prefetch_kernel<NT, kSwiGLU, bf16, kU>, inter / 8, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, inter);
+    }
+    if (mode == kSquaredReLU) {
+        if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+        return launch_pdl(gemm_skinny_wide_prefetch_kernel<NT, kSquaredReLU, bf16, kU>, N / kRows, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
     }
     if (out_dtype == PB_BF16)
         return launch_pdl(gemm_skinny_wide_prefetch_kernel<NT, kPlain, bf16, kU>, N / kRows, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
@@ -664,6 +675,10 @@ int launch_u(int mode, int out_dtype, const void* x, const void* w, void* out, i
         const GatedInter inter = gating_now(N / 2);
         if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
         return launch_pdl(gemm_skinny_kernel<NT, kSwiGLU, bf16, kUnroll>, inter / 8, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, inter);
+    }
+    if (mode == kSquaredReLU) {
+        if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+        return launch_pdl(gemm_skinny_kernel<NT, kSquaredReLU, bf16, kUnroll>, N / kRows, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
     }
     if (out_dtype == PB_BF16)
         return launch_pdl(gemm_skinny_kernel<NT, kPlain, bf16, kUnroll>, N / kRows, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
@@ -700,6 +715,10 @@ int launch(int mode, int out_dtype, const void* x, const void* w, void* out, int
             if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
             return launch_pdl(gemm_skinny_tall_kernel<kSwiGLU, bf16>, tiles / 2, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, N / 2);
         }
+        if (mode == kSquaredReLU) {
+            if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+            return launch_pdl(gemm_skinny_tall_kernel<kSquaredReLU, bf16>, tiles / 2, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
+        }
         if (out_dtype == PB_BF16)
             return launch_pdl(gemm_skinny_tall_kernel<kPlain, bf16>, tiles / 2, kWarps * 32, 0, stream, xp, wp, (bf16*)out, M, N, K, 0);
         return launch_pdl(gemm_skinny_tall_kernel<kPlain, float>, tiles / 2, kWarps * 32, 0, stream, xp, wp, (float*)out, M, N, K, 0);
@@ -714,7 +733,7 @@ int launch(int mode, int out_dtype, const void* x, const void* w, void* out, int
 PB_EXPORT int pb_gemm_skinny_supported(int mode, int M, int N, int K) {
     if (M <= 0 || M > 16 || K <= 0 || K % kBlockK) return 0;
     if (mode == kSwiGLU) return (N % 16 == 0) ? 1 : 0;       // N = 2 * inter, inter % 8 == 0
-    if (mode != kPlain) return 0;
+    if (mode != kPlain && mode != kSquaredReLU) return 0;
     return (N % kRows == 0) ? 1 : 0;
 }
 
@@ -789,7 +808,8 @@ PB_EXPORT int pb_gemm_skinny_scaled(int mode, const void* y, const void* w, void
 }
 
 // mode 0: out[M, N] (out_dtype bfloat16 or float32).  mode 1: W = [gate rows; up rows] with N = 2 * inter,
-// out[M, inter] = silu(x Wg^T) * (x Wu^T) in bfloat16.  x, W bfloat16, 16-byte aligned.
+// out[M, inter] = silu(x Wg^T) * (x Wu^T) in bfloat16.  mode 2: out[M, N] = max(x W^T, 0)^2 in bfloat16.  x, W bfloat16,
+// 16-byte aligned.
 PB_EXPORT int pb_gemm_skinny(int mode, int out_dtype, const void* x, const void* w, void* out, int M, int N, int K,
                              cudaStream_t stream) {
     if (!pb_gemm_skinny_supported(mode, M, N, K)) return PB_ERR_BAD_SIZE;

@@ -16,7 +16,8 @@
 //                        other accumulator with the next tile.
 // Epilogues: plain (bfloat16 or float32), or SwiGLU: the 256 columns are 128 gate features and
 // the 128 up features that belong to them (two TMA boxes from the two halves of the fused
-// weight), and silu(gate) * up is written, so the [M, 2I] intermediate never exists.
+// weight), and silu(gate) * up is written, so the [M, 2I] intermediate never exists; or the plain product's squared ReLU,
+// max(., 0)^2.
 //
 // Rows of x or W beyond the matrix and the tail of K are zero-filled by TMA; stores are
 // guarded.  Every wait is bounded by a clock limit: a block that gives up sets an error word
@@ -45,7 +46,7 @@ constexpr int kBBytes = kBN * kBK * 2;           // 32 KB
 constexpr int kStageBytes = kABytes + kBBytes;
 constexpr int kSmemBytes = kStages * kStageBytes + 1024 /* alignment slack */ + 256 /* barriers */;
 
-enum { kPlain = 0, kSwiGLU = 1 };
+enum { kPlain = 0, kSwiGLU = 1, kSquaredReLU = 2 };      // kSquaredReLU: the plain product's tiles, max(., 0)^2 on the way out
 
 __device__ unsigned int g_tc5_error = 0;          // 0 = fine; else 1 + the role that gave up
 
@@ -263,7 +264,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
                     tmem_ld32(lane_base + c, v);
                     float f[32];
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]);
+                    for (int i = 0; i < 32; ++i) f[i] = MODE == kSquaredReLU ? squared_relu(__uint_as_float(v[i])) : __uint_as_float(v[i]);
                     if (row < M && n0 + c < N) store32(out + (size_t)row * N + n0 + c, f, N - (n0 + c));
                 }
             }
@@ -402,7 +403,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                     tmem_ld32(lane_base + c, v);
                     float f[32];
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]);
+                    for (int i = 0; i < 32; ++i) f[i] = MODE == kSquaredReLU ? squared_relu(__uint_as_float(v[i])) : __uint_as_float(v[i]);
                     if (row < M && n0 + c < N) store32(out + (size_t)row * N + n0 + c, f, N - (n0 + c));
                 }
             }
@@ -552,7 +553,7 @@ gemm_tcgen05_grouped_kernel(const __grid_constant__ CUtensorMap map_x, const __g
                     tmem_ld32(lane_base + c, v);
                     float f[32];
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) f[i] = __uint_as_float(v[i]);
+                    for (int i = 0; i < 32; ++i) f[i] = MODE == kSquaredReLU ? squared_relu(__uint_as_float(v[i])) : __uint_as_float(v[i]);
                     if (row < M && n0 + c < N) store32(out + (size_t)row * N + n0 + c, f, N - (n0 + c));
                 }
             }
@@ -650,7 +651,7 @@ int launch(const CUtensorMap& mx, const CUtensorMap& mw, void* out, int M, int N
 PB_EXPORT int pb_gemm_tcgen05_supported(int mode, int M, int N, int K) {
     if (M <= 0 || N <= 0 || K <= 0 || (K % 8)) return 0;
     if (mode == kSwiGLU) return (N % 2 == 0) ? 1 : 0;
-    return mode == kPlain ? 1 : 0;
+    return (mode == kPlain || mode == kSquaredReLU) ? 1 : 0;
 }
 
 // The error word of the kernel's bounded waits (0 = no block ever gave up); reading it synchronises.
@@ -693,7 +694,8 @@ PB_EXPORT int pb_gemm_tcgen05_wait_selftest(cudaStream_t stream) {
 }
 
 // mode 0: out[M, N] = x W^T (out_dtype bfloat16 or float32).  mode 1: W = [gate rows; up rows], N = 2 * inter,
-// out[M, inter] = silu(x Wg^T) * (x Wu^T) in bfloat16.  x [M, K] and W [N, K] bfloat16, 16-byte aligned.
+// out[M, inter] = silu(x Wg^T) * (x Wu^T) in bfloat16.  mode 2: out[M, N] = max(x W^T, 0)^2 in bfloat16.  x [M, K] and
+// W [N, K] bfloat16, 16-byte aligned.
 PB_EXPORT int pb_gemm_tcgen05(int mode, int out_dtype, const void* x, const void* w, void* out, int M, int N, int K,
                               cudaStream_t stream) {
     if (!pb_gemm_tcgen05_supported(mode, M, N, K)) return PB_ERR_BAD_SIZE;
@@ -711,6 +713,10 @@ PB_EXPORT int pb_gemm_tcgen05(int mode, int out_dtype, const void* x, const void
         return launch<kSwiGLU, bf16>(mx, mw, out, M, N, K, inter, m_tiles, (inter + kBN / 2 - 1) / (kBN / 2), stream);
     }
     const int n_tiles = (N + kBN - 1) / kBN;
+    if (mode == kSquaredReLU) {
+        if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+        return launch<kSquaredReLU, bf16>(mx, mw, out, M, N, K, 0, m_tiles, n_tiles, stream);
+    }
     if (out_dtype == PB_BF16) return launch<kPlain, bf16>(mx, mw, out, M, N, K, 0, m_tiles, n_tiles, stream);
     return launch<kPlain, float>(mx, mw, out, M, N, K, 0, m_tiles, n_tiles, stream);
 }
@@ -719,8 +725,9 @@ PB_EXPORT int pb_gemm_tcgen05(int mode, int out_dtype, const void* x, const void
 // The grouped product (see gemm_tcgen05_grouped_kernel): x [P, K] rows sorted by group, W [n_groups * w_rows, K] the groups'
 // matrices one behind the other, bfloat16.  mode 0: w_rows = N, out [P, N] (out_dtype bfloat16 or float32) = x W[group]^T.
 // mode 1: w_rows = 2 * inter (gate rows, then up rows), out [P, inter] bfloat16 = the gated unit (limit <= 0: none).
+// mode 2: w_rows = N, out [P, N] bfloat16 = max(x W[group]^T, 0)^2.
 // offsets [n_groups + 1], tile_group / tile_row0 [max_row_tiles], meta[0] = tiles listed: device arrays.
-// pair_scale (mode 1, or null): row r's gate and up sums are multiplied by pair_scale[row_pair[r]] before the gating.
+// pair_scale (mode 1 only, or null): row r's gate and up sums are multiplied by pair_scale[row_pair[r]] before the gating.
 PB_EXPORT int pb_gemm_tcgen05_grouped(int mode, int out_dtype, const void* x, const void* w, void* out, int P, int N, int K,
                                       int n_groups, const int* offsets, const int* tile_group, const int* tile_row0, const int* meta,
                                       int max_row_tiles, float limit, float alpha, float shift, const int* row_pair,
@@ -756,6 +763,10 @@ PB_EXPORT int pb_gemm_tcgen05_grouped(int mode, int out_dtype, const void* x, co
         PB_GROUPED(kSwiGLU, bf16, inter, ((int)inter + kBN / 2 - 1) / (kBN / 2))
     }
     const int n_tiles = (N + kBN - 1) / kBN;
+    if (mode == kSquaredReLU) {
+        if (out_dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+        PB_GROUPED(kSquaredReLU, bf16, GatedInter(0), n_tiles)
+    }
     if (out_dtype == PB_BF16) PB_GROUPED(kPlain, bf16, GatedInter(0), n_tiles)
     PB_GROUPED(kPlain, float, GatedInter(0), n_tiles)
 #undef PB_GROUPED

@@ -13,6 +13,9 @@
 //                    the token's cache slot (and, where asked, to contiguous rows for the expanded form);
 //                    rotation of every head's rotated query part into its float32 query row
 //                    ([q_abs | q_rot], or [q_plain | q_rot] for the expanded form).
+//   latent_norms     the first half of that for layers whose queries come out of a latent of their own: the RMS norm of the
+//                    queries' latent (float32, one rounding) to contiguous rows, and, where the layer owns its cache rows, the
+//                    latent part and the rotated key part as above.  One block per token and latent.
 //   latent_expand_keys, sigmoid_gate: the expanded form's key rows [plain | shared rotated part], and its output gate.
 // The rotation pairs neighbours: (x[2i], x[2i+1]) turns by the angle of table column i; dimensions
 // beyond the rotated ones pass unchanged.
@@ -137,6 +140,69 @@ struct PrepareShape {
     float eps;
 };
 
+// One token's row of the down projection: its latent part normed and its rotated part turned, to the token's cache slot and
+// (where asked) to contiguous rows.
+template <typename T>
+__device__ __forceinline__ void cache_latent_row(const T* __restrict__ x, const float* __restrict__ norm_w, const float* __restrict__ ct,
+                                                 const float* __restrict__ st, const int* __restrict__ slots, T* __restrict__ pool,
+                                                 T* __restrict__ latent_out, T* __restrict__ rot_out, int t, int rank, int rot_dim,
+                                                 int rot_dims, int page_size, float eps, float* scratch, const PoolBounds& bounds) {
+    const int half = rot_dims >> 1;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_float(x[i]); ss += v * v; }
+    ss = block_sum(ss, scratch);
+    const float inv = rsqrtf(ss / (float)rank + eps);
+    const int slot = slots[t];
+    const bool cached = slot >= 0 && slot_ok(slot, page_size, bounds);
+    T* dst = pool + (size_t)(cached ? slot : 0) * (rank + rot_dim);   // [pages, 1, page, rank + rot_dim]: slot = page * page_size + offset
+    T* lat = latent_out ? latent_out + (size_t)t * rank : nullptr;
+    T* rot = rot_out ? rot_out + (size_t)t * rot_dim : nullptr;
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+        const T v = from_float<T>(to_float(x[i]) * inv * norm_w[i]);
+        if (cached) dst[i] = v;
+        if (lat) lat[i] = v;
+    }
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float u = to_float(x[rank + 2 * i]), v = to_float(x[rank + 2 * i + 1]);
+        const T a = from_float<T>(u * ct[i] - v * st[i]), b = from_float<T>(v * ct[i] + u * st[i]);
+        if (cached) { dst[rank + 2 * i] = a; dst[rank + 2 * i + 1] = b; }
+        if (rot) { rot[2 * i] = a; rot[2 * i + 1] = b; }
+    }
+    for (int i = rot_dims + threadIdx.x; i < rot_dim; i += blockDim.x) {
+        if (cached) dst[rank + i] = x[rank + i];
+        if (rot) rot[i] = x[rank + i];
+    }
+}
+
+struct NormsShape {
+    int q_rank, rank, rot_dim, rot_dims, page_size;
+    long q_tok, down_tok;
+    float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_norms_kernel(const T* __restrict__ q_lat, const float* __restrict__ q_norm_w, T* __restrict__ q_out, const T* __restrict__ down,
+                    const float* __restrict__ norm_w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                    const int* __restrict__ slots, T* __restrict__ pool, T* __restrict__ latent_out, T* __restrict__ rot_out,
+                    const NormsShape sh, const PoolBounds bounds) {
+    pdl_wait();         // may have come onto the SMs while the product before it was ending: nothing is touched before that one is done
+    __shared__ float scratch[32];
+    const int t = blockIdx.x;
+    if (blockIdx.y == 0) {
+        const T* x = q_lat + (size_t)t * sh.q_tok;
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < sh.q_rank; i += blockDim.x) { const float v = to_float(x[i]); ss += v * v; }
+        const float inv = rsqrtf(block_sum(ss, scratch) / (float)sh.q_rank + sh.eps);
+        for (int i = threadIdx.x; i < sh.q_rank; i += blockDim.x)
+            q_out[(size_t)t * sh.q_rank + i] = from_float<T>(to_float(x[i]) * inv * q_norm_w[i]);
+        return;
+    }
+    const int half = sh.rot_dims >> 1;
+    cache_latent_row(down + (size_t)t * sh.down_tok, norm_w, cos_t + (size_t)t * half, sin_t + (size_t)t * half, slots, pool, latent_out,
+                     rot_out, t, sh.rank, sh.rot_dim, sh.rot_dims, sh.page_size, sh.eps, scratch, bounds);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_prepare_kernel(const T* __restrict__ q, const T* __restrict__ down, const float* __restrict__ norm_w,
@@ -145,36 +211,12 @@ latent_prepare_kernel(const T* __restrict__ q, const T* __restrict__ down, const
                       const PrepareShape sh, const PoolBounds bounds) {
     __shared__ float scratch[32];
     const int t = blockIdx.x;
-    const int rank = sh.rank, rot_dim = sh.rot_dim, half = sh.rot_dims >> 1;
+    const int rot_dim = sh.rot_dim, half = sh.rot_dims >> 1;
     const float* ct = cos_t + (size_t)t * half;
     const float* st = sin_t + (size_t)t * half;
-    if (down != nullptr) {                      // uniform over the block
-        const T* x = down + (size_t)t * sh.down_tok;
-        float ss = 0.0f;
-        for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_float(x[i]); ss += v * v; }
-        ss = block_sum(ss, scratch);
-        const float inv = rsqrtf(ss / (float)rank + sh.eps);
-        const int slot = slots[t];
-        const bool cached = slot >= 0 && slot_ok(slot, sh.page_size, bounds);
-        T* dst = pool + (size_t)(cached ? slot : 0) * (rank + rot_dim);   // [pages, 1, page, rank + rot_dim]: slot = page * page_size + offset
-        T* lat = latent_out ? latent_out + (size_t)t * rank : nullptr;
-        T* rot = rot_out ? rot_out + (size_t)t * rot_dim : nullptr;
-        for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-            const T v = from_float<T>(to_float(x[i]) * inv * norm_w[i]);
-            if (cached) dst[i] = v;
-            if (lat) lat[i] = v;
-        }
-        for (int i = threadIdx.x; i < half; i += blockDim.x) {
-            const float u = to_float(x[rank + 2 * i]), v = to_float(x[rank + 2 * i + 1]);
-            const T a = from_float<T>(u * ct[i] - v * st[i]), b = from_float<T>(v * ct[i] + u * st[i]);
-            if (cached) { dst[rank + 2 * i] = a; dst[rank + 2 * i + 1] = b; }
-            if (rot) { rot[2 * i] = a; rot[2 * i + 1] = b; }
-        }
-        for (int i = sh.rot_dims + threadIdx.x; i < rot_dim; i += blockDim.x) {
-            if (cached) dst[rank + i] = x[rank + i];
-            if (rot) rot[i] = x[rank + i];
-        }
-    }
+    if (down != nullptr)                        // uniform over the block
+        cache_latent_row(down + (size_t)t * sh.down_tok, norm_w, ct, st, slots, pool, latent_out, rot_out, t, sh.rank, rot_dim, sh.rot_dims,
+                         sh.page_size, sh.eps, scratch, bounds);
     const int per_head = sh.dim + rot_dim, H = sh.H;
     for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
         const int h = i / half, j = i % half;
@@ -277,6 +319,28 @@ PB_EXPORT int pb_latent_prepare(int dtype, const void* q, long q_tok, const void
                                                                     pb::pool_bounds_now());
     else return PB_ERR_BAD_DTYPE;
     return launch_status();
+}
+
+// q_lat: rows of q_rank at n * q_tok, normed with q_norm_w (float32 [q_rank]) into q_out [N, q_rank].  down (may be null) and what
+// becomes of it: as in pb_latent_prepare.
+PB_EXPORT int pb_latent_norms(int dtype, const void* q_lat, long q_tok, const float* q_norm_w, void* q_out, const void* down, long down_tok,
+                              const float* norm_w, float eps, const float* cos_t, const float* sin_t, const int* slots, void* pool,
+                              void* latent_out, void* rot_out, int N, int q_rank, int rank, int rot_dim, int rot_dims, int page_size,
+                              cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (q_rank <= 0 || rank <= 0 || rot_dim < 0 || rot_dims < 0 || rot_dims > rot_dim || rot_dims % 2 || page_size <= 0) return PB_ERR_BAD_SIZE;
+    if (down != nullptr && (norm_w == nullptr || slots == nullptr || pool == nullptr)) return PB_ERR_BAD_SIZE;
+    const NormsShape sh{q_rank, rank, rot_dim, rot_dims, page_size, q_tok, down_tok, eps};
+    const dim3 grid(N, down != nullptr ? 2 : 1);
+    if (dtype == PB_F32)
+        return launch_pdl(latent_norms_kernel<float>, grid, dim3(128), 0, stream, (const float*)q_lat, q_norm_w, (float*)q_out,
+                          (const float*)down, norm_w, cos_t, sin_t, slots, (float*)pool, (float*)latent_out, (float*)rot_out, sh,
+                          pb::pool_bounds_now());
+    if (dtype == PB_BF16)
+        return launch_pdl(latent_norms_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, (const __nv_bfloat16*)q_lat, q_norm_w,
+                          (__nv_bfloat16*)q_out, (const __nv_bfloat16*)down, norm_w, cos_t, sin_t, slots, (__nv_bfloat16*)pool,
+                          (__nv_bfloat16*)latent_out, (__nv_bfloat16*)rot_out, sh, pb::pool_bounds_now());
+    return PB_ERR_BAD_DTYPE;
 }
 
 PB_EXPORT int pb_latent_expand_keys(int dtype, const void* plain, const void* shared, void* keys, int N, int H, int dim, int rot_dim,

@@ -5,13 +5,19 @@
 //                  chosen s * scale.  ids int32 [N, top] in descending order of s, weights float32 [N, top].
 //                  With `softmax` the scores are s = softmax(z) over all experts instead, and a renormalised weight is
 //                  s / (sum of the chosen s + renorm_eps) * scale.
+//                  With `correction` (float32 [E]) the choice goes by s + correction[e], the weights by s alone.  With
+//                  keep_groups < n_groups the experts form n_groups groups of neighbours of equal size, a group counts as its
+//                  best choice score, and only experts of the keep_groups best groups can be chosen.
 //   moe_gate_up    for every (token, chosen expert): g = W_gate[e] h, u = W_up[e] h (float32 sums), the gated unit
 //                  out = g' * sigmoid(alpha * g') * (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit),
 //                  one rounding on store: act [N * top, ff].  Weights [E, 2 ff, width]: an expert's gate rows, then
 //                  its up rows.
 //   moe_down       out[n] = add[n] + sum over the chosen experts, in the order of ids, of weight * (W_down[e] act[n, slot]);
 //                  float32 sums, one rounding on store.  Weights [E, width, ff].  `add` (optional): what a shared
-//                  expert contributed.
+//                  expert contributed.  Ids from n_real on are identity experts without weights: they contribute
+//                  weight * h[n].
+//   moe_up         ungated experts: act [N * top, ff] = max(W_up[e] h, 0)^2 for every (token, chosen expert) with e < n_real;
+//                  weights [n_real, ff, width].
 // A warp owns one output element and walks the contraction in a fixed order, so a token's result does not depend on
 // what else is in the step.  These kernels read an expert's weights once per token that chose it: they are for steps
 // of a few tokens (and for the float32 engine); larger steps sort the tokens by expert and take the grouped product.
@@ -31,6 +37,13 @@ __device__ __forceinline__ void load_chunk(const __nv_bfloat16* p, float (&f)[8]
 #pragma unroll
     for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(u[i] << 16); f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u); }
 }
+// What the choice goes by besides the scores: a number added to each (or null), and how many of the groups of neighbours
+// the chosen experts may come from (keep >= n_groups: all).
+struct RouteChoice {
+    const float* correction;
+    int n_groups, keep;
+};
+
 constexpr int kRouteRows = 4;            // router rows a warp walks side by side: their loads are in flight together
 
 __device__ __forceinline__ void fma4(float& z, const float4& a, const float4& x) {
@@ -44,11 +57,14 @@ __device__ __forceinline__ void fma4(float& z, const float4& a, const float4& x)
 template <typename T, int TOK>
 __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, int* __restrict__ ids,
                                  float* __restrict__ weights, int n, int width, int n_experts, int top, float scale,
-                                 int renormalize, int n_extra, float* __restrict__ extra, int softmax, float renorm_eps) {
+                                 int renormalize, int n_extra, float* __restrict__ extra, int softmax, float renorm_eps,
+                                 const RouteChoice choice) {
     pdl_wait();
     extern __shared__ __align__(16) float smem[];
     float* x = smem;                                     // [TOK][width]
     float* s = smem + (size_t)TOK * width;               // [TOK][n_experts + n_extra]
+    float* picks = s + (size_t)TOK * (n_experts + n_extra);      // [TOK][n_experts]: the choice scores
+    float* bests = picks + (size_t)TOK * n_experts;      // [TOK][n_groups]: a group's best choice score
     const int n_rows = n_experts + n_extra;              // the rows behind the experts' compete for nothing: their sigmoids go to `extra`
     const int t0 = blockIdx.x * TOK, n_tok = min(TOK, n - t0);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -154,25 +170,46 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
         for (int e = lane; e < n_experts; e += 32) sk[e] = sk[e] / sum;
         __syncwarp();
     }
+    float* pick = picks + (size_t)warp * n_experts;
+    for (int e = lane; e < n_experts; e += 32) pick[e] = sk[e] + (choice.correction ? choice.correction[e] : 0.0f);
+    __syncwarp();
+    if (choice.keep < choice.n_groups) {                 // uniform over the grid
+        float* best = bests + (size_t)warp * choice.n_groups;
+        const int size = n_experts / choice.n_groups;
+        for (int g = lane; g < choice.n_groups; g += 32) {
+            float m = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, pick[e]);
+            best[g] = m;
+        }
+        __syncwarp();
+        for (int g = lane; g < choice.n_groups; g += 32) {
+            int ahead = 0;                               // groups in front of this one; among equals the lower index
+            for (int o = 0; o < choice.n_groups; ++o) ahead += best[o] > best[g] || (best[o] == best[g] && o < g);
+            if (ahead >= choice.keep)
+                for (int e = g * size; e < (g + 1) * size; ++e) pick[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float total = 0.0f;
     for (int c = 0; c < top; ++c) {
-        // the largest score left; among equals the lowest index
-        float best = -1.0f;
+        // the largest choice score left; among equals the lowest index
+        float best = -INFINITY;
         int arg = n_experts;
         for (int e = lane; e < n_experts; e += 32)
-            if (sk[e] > best) { best = sk[e]; arg = e; }
+            if (pick[e] > best) { best = pick[e]; arg = e; }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
             const float ob = __shfl_xor_sync(0xffffffffu, best, o);
             const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
+        arg = min(arg, n_experts - 1);       // (no score is a number: an id that exists all the same)
         if (lane == 0) {
             ids[t * top + c] = arg;
-            weights[t * top + c] = best;
-            sk[arg] = -2.0f;                 // taken
+            weights[t * top + c] = sk[arg];
+            pick[arg] = -INFINITY;           // taken
         }
-        total += best;
+        total += sk[arg];
         __syncwarp();
     }
     if (lane == 0) {
@@ -246,9 +283,27 @@ __global__ void moe_gate_up_kernel(const T* __restrict__ h, const T* __restrict_
 }
 
 template <typename T>
+__global__ void moe_up_kernel(const T* __restrict__ h, const T* __restrict__ w_up, const int* __restrict__ ids, T* __restrict__ act,
+                              int width, int ff, int top, int n_real) {
+    pdl_wait();
+    extern __shared__ __align__(16) float x[];             // [width]
+    const int pair = blockIdx.x, t = pair / top;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const int e = ids[pair];
+    if (e >= n_real) return;                               // an identity expert has nothing to compute
+    for (int i = threadIdx.x; i < width; i += blockDim.x) x[i] = to_float(h[(size_t)t * width + i]);
+    __syncthreads();
+    const T* w = w_up + (size_t)e * ff * width;
+    for (int j = blockIdx.y * warps + warp; j < ff; j += gridDim.y * warps) {
+        const float u = dot_row(w + (size_t)j * width, x, width, lane);
+        if (lane == 0) act[(size_t)pair * ff + j] = from_float<T>(squared_relu(u));
+    }
+}
+
+template <typename T>
 __global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__ w_down, const int* __restrict__ ids,
                                 const float* __restrict__ weights, const T* __restrict__ add, const float* __restrict__ add_scale,
-                                T* __restrict__ out, int width, int ff, int top) {
+                                T* __restrict__ out, int width, int ff, int top, const T* __restrict__ h, int n_real) {
     pdl_wait();
     extern __shared__ __align__(16) float y[];             // [top][ff]
     const int t = blockIdx.x;
@@ -259,6 +314,10 @@ __global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__
         float sum = add ? to_float(add[(size_t)t * width + c]) * (add_scale ? add_scale[t] : 1.0f) : 0.0f;
         for (int slot = 0; slot < top; ++slot) {
             const int e = ids[(size_t)t * top + slot];
+            if (h != nullptr && e >= n_real) {             // uniform over the block
+                sum = fmaf(weights ? weights[(size_t)t * top + slot] : 1.0f, to_float(h[(size_t)t * width + c]), sum);
+                continue;
+            }
             const float d = dot_row(w_down + ((size_t)e * width + c) * ff, y + (size_t)slot * ff, ff, lane);
             sum = fmaf(weights ? weights[(size_t)t * top + slot] : 1.0f, d, sum);
         }
@@ -268,8 +327,8 @@ __global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__
 
 template <typename T, int TOK>
 int launch_route(const void* h, const float* router, int* ids, float* weights, int n, int width, int n_experts, int top, float scale,
-                 int renormalize, int n_extra, float* extra, int softmax, float renorm_eps, cudaStream_t stream) {
-    const size_t smem = sizeof(float) * TOK * ((size_t)width + n_experts + n_extra);
+                 int renormalize, int n_extra, float* extra, int softmax, float renorm_eps, const RouteChoice& choice, cudaStream_t stream) {
+    const size_t smem = sizeof(float) * TOK * ((size_t)width + 2 * n_experts + n_extra + choice.n_groups);
     if (smem > 200 * 1024) return PB_ERR_TOO_LARGE;
     static size_t allowed = 48 * 1024;
     if (smem > allowed) {
@@ -281,16 +340,16 @@ int launch_route(const void* h, const float* router, int* ids, float* weights, i
     if (warps > 16) warps = 16;
     if (warps < TOK) warps = TOK;                                         // warp k picks for token k
     return launch_pdl(moe_route_kernel<T, TOK>, dim3((n + TOK - 1) / TOK), dim3(32 * warps), smem, stream, (const T*)h, router, ids,
-                      weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps);
+                      weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, choice);
 }
 
 template <typename T>
 int dispatch_route(const void* h, const float* router, int* ids, float* weights, int n, int width, int n_experts, int top, float scale,
-                   int renormalize, int n_extra, float* extra, int softmax, float renorm_eps, cudaStream_t stream) {
+                   int renormalize, int n_extra, float* extra, int softmax, float renorm_eps, const RouteChoice& choice, cudaStream_t stream) {
     // tokens a block shares the router's rows among: one where the step is a few tokens (their blocks run side by side),
     // eight where their float32 rows leave room for three blocks on a SM, else four
-    const size_t row = sizeof(float) * ((size_t)width + n_experts + n_extra);
-#define PB_ROUTE(TOK) return launch_route<T, TOK>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, stream)
+    const size_t row = sizeof(float) * ((size_t)width + 2 * n_experts + n_extra + choice.n_groups);
+#define PB_ROUTE(TOK) return launch_route<T, TOK>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, choice, stream)
     if (n <= 16) PB_ROUTE(1);
     if (8 * row <= 72 * 1024) PB_ROUTE(8);
     PB_ROUTE(4);
@@ -299,15 +358,21 @@ int dispatch_route(const void* h, const float* router, int* ids, float* weights,
 
 }  // namespace
 
+// correction (float32 [n_experts] or null) joins the scores for the choice; n_groups groups of neighbours, keep_groups of them
+// open to the choice (1, 1: all experts).
 // router [n_experts + n_extra, width]: the rows behind the experts' are scored too (sigmoid) and go to extra [n, n_extra].
 PB_EXPORT int pb_moe_route(int dtype, const void* h, const float* router, int* ids, float* weights, int n, int width, int n_experts,
                            int top, float scale, int renormalize, int n_extra, float* extra, int softmax, float renorm_eps,
-                           cudaStream_t stream) {
+                           const float* correction, int n_groups, int keep_groups, cudaStream_t stream) {
     if (n <= 0) return 0;
+    if (n_groups <= 0 || keep_groups <= 0 || n_experts % n_groups ||
+        (keep_groups < n_groups && (long)keep_groups * (n_experts / n_groups) < top))
+        return PB_ERR_BAD_SIZE;
+    const RouteChoice choice{correction, n_groups, keep_groups};
     if (width <= 0 || n_experts <= 0 || top <= 0 || top > n_experts || n_extra < 0 || (n_extra > 0 && extra == nullptr)) return PB_ERR_BAD_SIZE;
-    if (dtype == PB_F32) return dispatch_route<float>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, stream);
+    if (dtype == PB_F32) return dispatch_route<float>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, choice, stream);
     if (dtype == PB_BF16)
-        return dispatch_route<__nv_bfloat16>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, stream);
+        return dispatch_route<__nv_bfloat16>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, choice, stream);
     return PB_ERR_BAD_DTYPE;
 }
 
@@ -332,22 +397,55 @@ PB_EXPORT int pb_moe_gate_up(int dtype, const void* h, const void* w_gate_up, co
     return PB_ERR_BAD_DTYPE;
 }
 
+// Ungated experts: act [n * top, ff] = max(w_up[e] h, 0)^2, w_up [n_real, ff, width]; pairs with ids >= n_real are left out.
+PB_EXPORT int pb_moe_up(int dtype, const void* h, const void* w_up, const int* ids, void* act, int n, int width, int ff, int top,
+                        int n_real, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (width <= 0 || ff <= 0 || top <= 0 || n_real <= 0) return PB_ERR_BAD_SIZE;
+    const size_t smem = sizeof(float) * (size_t)width;
+    if (smem > 48 * 1024) return PB_ERR_TOO_LARGE;
+    const int warps = 8;
+    int by = (ff + warps - 1) / warps;
+    if (by > 64) by = 64;
+    dim3 grid(n * top, by);
+    if (dtype == PB_F32)
+        return launch_pdl(moe_up_kernel<float>, grid, dim3(warps * 32), smem, stream, (const float*)h, (const float*)w_up, ids, (float*)act,
+                          width, ff, top, n_real);
+    if (dtype == PB_BF16)
+        return launch_pdl(moe_up_kernel<__nv_bfloat16>, grid, dim3(warps * 32), smem, stream, (const __nv_bfloat16*)h,
+                          (const __nv_bfloat16*)w_up, ids, (__nv_bfloat16*)act, width, ff, top, n_real);
+    return PB_ERR_BAD_DTYPE;
+}
+
 // weights null: every pair counts once (its weight went into the expert's input); add_scale (float32 [n] or null) multiplies `add`.
+// h [n, width] (or null: no identity experts): what a pair with an id >= n_real contributes, times its weight.
 PB_EXPORT int pb_moe_down(int dtype, const void* act, const void* w_down, const int* ids, const float* weights, const void* add,
-                          const float* add_scale, void* out, int n, int width, int ff, int top, cudaStream_t stream) {
+                          const float* add_scale, void* out, int n, int width, int ff, int top, const void* h, int n_real,
+                          cudaStream_t stream) {
     if (n <= 0) return 0;
     if (width <= 0 || ff <= 0 || top <= 0) return PB_ERR_BAD_SIZE;
     const size_t smem = sizeof(float) * (size_t)top * ff;
-    if (smem > 48 * 1024) return PB_ERR_TOO_LARGE;
+    if (smem > 200 * 1024) return PB_ERR_TOO_LARGE;
+    if (dtype != PB_F32 && dtype != PB_BF16) return PB_ERR_BAD_DTYPE;
+    static size_t allowed[2] = {48 * 1024, 48 * 1024};
+    size_t& mine = allowed[dtype == PB_BF16];
+    if (smem > mine) {
+        const cudaError_t ce = dtype == PB_F32
+            ? cudaFuncSetAttribute(moe_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
+            : cudaFuncSetAttribute(moe_down_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (ce != cudaSuccess) return (int)ce;
+        mine = smem;
+    }
     const int warps = 8;
     int by = (width + warps - 1) / warps;
     if (by > 64) by = 64;
     dim3 grid(n, by);
     if (dtype == PB_F32)
         return launch_pdl(moe_down_kernel<float>, grid, dim3(warps * 32), smem, stream, (const float*)act, (const float*)w_down, ids,
-                          weights, (const float*)add, add_scale, (float*)out, width, ff, top);
+                          weights, (const float*)add, add_scale, (float*)out, width, ff, top, (const float*)h, n_real);
     if (dtype == PB_BF16)
         return launch_pdl(moe_down_kernel<__nv_bfloat16>, grid, dim3(warps * 32), smem, stream, (const __nv_bfloat16*)act,
-                          (const __nv_bfloat16*)w_down, ids, weights, (const __nv_bfloat16*)add, add_scale, (__nv_bfloat16*)out, width, ff, top);
+                          (const __nv_bfloat16*)w_down, ids, weights, (const __nv_bfloat16*)add, add_scale, (__nv_bfloat16*)out, width, ff, top,
+                          (const __nv_bfloat16*)h, n_real);
     return PB_ERR_BAD_DTYPE;
 }

@@ -6,6 +6,7 @@
 //                   tile_row0[t] .. of expert tile_expert[t]; meta[0] = number of tiles.  One block; nothing returns to the host.
 //   moe_grouped     mode 0: act[sorted row] = gated(h[token] Wg[e]^T, h[token] Wu[e]^T)   (rows gathered by pair / top)
 //                   mode 1: y[sorted row] (float32) = act[sorted row] W_down[e]^T
+//                   mode 2: act[sorted row] = max(h[token] Wup[e]^T, 0)^2                  (ungated experts)
 //                   mma.sync m16n8k16, bfloat16 operands, float32 accumulators; tiles of 128 rows x 64 output columns
 //                   (mode 0: 64 gate and the 64 up columns that go with them), K in steps of 64 through a three-stage cp.async
 //                   pipeline.  The grid has as many row tiles as the worst case needs; blocks beyond meta[0] return at once.
@@ -14,6 +15,8 @@
 // Where the sizes allow it (contraction widths that are multiples of 8, as for every tcgen05 product of this library) the two
 // products run on the grouped form of the tcgen05 kernel instead (pb_gemm_tcgen05_grouped: TMA, tensor memory, the same tile
 // list), with the tokens' rows gathered into sorted order first (moe_gather_rows); PULSAR_MOE_TCGEN05=0 keeps mma.sync.
+// Ids from n_experts on are identity experts: such a pair is in no group (its place is -1) and moe_combine takes the token's
+// own row of h for it.
 // A row's result depends on that row and its expert's weights alone, so the order of the pairs inside an expert (which the
 // sort leaves to the atomics) does not show in the output.
 #include "mma_common.cuh"
@@ -34,7 +37,8 @@ __global__ void moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int n_
     int* cursor = sh + n_experts;
     for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
     __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&counts[ids[p]], 1);
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
+        if (ids[p] < n_experts) atomicAdd(&counts[ids[p]], 1);
     __syncthreads();
     if (threadIdx.x == 0) {
         int at = 0, tiles = 0;
@@ -53,6 +57,10 @@ __global__ void moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int n_
     }
     __syncthreads();
     for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
+        if (ids[p] >= n_experts) {
+            place[p] = -1;
+            continue;
+        }
         const int at = atomicAdd(&cursor[ids[p]], 1);
         sorted[at] = p;
         place[p] = at;
@@ -60,16 +68,17 @@ __global__ void moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int n_
 }
 
 // rows[at] = h[sorted[at] / top]: the tokens' rows in the order of the sorted pairs, 16 bytes a thread.
-__global__ void moe_gather_rows_kernel(const bf16* __restrict__ h, const int* __restrict__ sorted, bf16* __restrict__ rows, int width,
-                                       int top) {
+__global__ void moe_gather_rows_kernel(const bf16* __restrict__ h, const int* __restrict__ sorted, const int* __restrict__ n_sorted,
+                                       bf16* __restrict__ rows, int width, int top) {
     pdl_wait();
     const int at = blockIdx.x;
+    if (at >= *n_sorted) return;                       // fewer sorted pairs than pairs where some are identity experts'
     const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)(sorted[at] / top) * width);
     uint4* dst = reinterpret_cast<uint4*>(rows + (size_t)at * width);
     for (int i = threadIdx.x; i < width / 8; i += blockDim.x) dst[i] = src[i];
 }
 
-// MODE 0: gate/up with the gating; MODE 1: down.  Eight warps, four along the rows and two along the columns: a warp owns
+// MODE 0: gate/up with the gating; MODE 1: down; MODE 2: up with the squared ReLU.  Eight warps, four along the rows and two along the columns: a warp owns
 // 32 rows x 32 output columns (mode 0: 32 gate columns and the 32 up columns that go with them).
 template <int MODE>
 __global__ void __launch_bounds__(kThreads)
@@ -93,7 +102,7 @@ moe_grouped_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, const
     const int warp_m = warp >> 1, warp_n = warp & 1;
     if (tid < kBM) {
         int r = -1;
-        if (tid < rows) r = MODE == 0 ? sorted[row0 + tid] / top : row0 + tid;
+        if (tid < rows) r = MODE != 1 ? sorted[row0 + tid] / top : row0 + tid;
         src_row[tid] = r;
     }
     __syncthreads();
@@ -183,6 +192,14 @@ moe_grouped_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, const
                         if (col + 1 < n_out) dst[col + 1] = __float2bfloat16_rn(v1);
                     }
                 }
+            } else if (MODE == 2) {
+                bf16* dst = act_out + (size_t)(row0 + r) * n_out;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int col = n0 + warp_n * 32 + j * 8 + 2 * t;
+                    if (col < n_out) dst[col] = __float2bfloat16_rn(squared_relu(acc[mi][j][2 * half]));
+                    if (col + 1 < n_out) dst[col + 1] = __float2bfloat16_rn(squared_relu(acc[mi][j][2 * half + 1]));
+                }
             } else {
                 float* dst = y_out + (size_t)(row0 + r) * n_out;
 #pragma unroll
@@ -199,14 +216,16 @@ moe_grouped_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, const
 }
 
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights,
-                                   const bf16* __restrict__ add, const float* __restrict__ add_scale, bf16* __restrict__ out, int width,
-                                   int top, size_t total) {
+                                   const bf16* __restrict__ add, const float* __restrict__ add_scale, const bf16* __restrict__ h,
+                                   bf16* __restrict__ out, int width, int top, size_t total) {
     pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t n = i / width, c = i % width;
         float sum = add ? __bfloat162float(add[i]) * (add_scale ? add_scale[n] : 1.0f) : 0.0f;
-        for (int slot = 0; slot < top; ++slot)
-            sum = fmaf(weights ? weights[n * top + slot] : 1.0f, y[(size_t)place[n * top + slot] * width + c], sum);
+        for (int slot = 0; slot < top; ++slot) {
+            const int at = place[n * top + slot];
+            sum = fmaf(weights ? weights[n * top + slot] : 1.0f, at < 0 ? __bfloat162float(h[i]) : y[(size_t)at * width + c], sum);
+        }
         out[i] = __float2bfloat16_rn(sum);
     }
 }
@@ -224,7 +243,7 @@ PB_EXPORT int pb_moe_grouped_supported(int width, int ff, int n_experts) {
     return (width > 0 && ff > 0 && width % 8 == 0 && ff % 8 == 0 && n_experts > 0 && n_experts <= 4096) ? 1 : 0;
 }
 
-// h [n, width], w_gate_up [E, 2 ff, width], w_down [E, width, ff], add [n, width] or null, out [n, width]: bfloat16;
+// h [n, width], w_gate_up [E, 2 ff, width] ([E, ff, width] ungated), w_down [E, width, ff], add [n, width] or null, out [n, width]: bfloat16;
 // ids int32 [n, top], weights float32 [n, top]; act bfloat16 [n * top, ff] and y float32 [n * top, width] scratch;
 // work: int32 scratch of pb_moe_grouped_workspace(n, top, E) elements.  limit <= 0: no clamp.  gathered: bfloat16
 // [n * top, width] scratch for the tcgen05 form, or null for the mma.sync form.
@@ -236,13 +255,15 @@ PB_EXPORT int pb_gemm_tcgen05_grouped(int mode, int out_dtype, const void* x, co
 PB_EXPORT int pb_moe_grouped(const void* h, const void* w_gate_up, const void* w_down, const int* ids, const float* weights,
                              const void* add, void* act, float* y, void* out, int* work, void* gathered, int n, int width, int ff,
                              int n_experts, int top, float limit, float alpha, float shift, int weight_input, const float* add_scale,
-                             cudaStream_t stream) {
+                             int ungated, int n_identity, cudaStream_t stream) {
     if (n <= 0) return 0;
+    if (ungated && weight_input) return PB_ERR_BAD_SIZE;
+    // ungated: w_gate_up is [E, ff, width] and the unit max(., 0)^2.  n_identity: ids may go up to n_experts + n_identity - 1.
     // weight_input: a pair's weight multiplies its expert's input (in the gate/up epilogue: W (w h) = w (W h)) and the sum
     // over a token's experts takes every pair once; add_scale (float32 [n] or null) multiplies `add`.
     const float* in_weights = weight_input ? weights : nullptr;
     const float* out_weights = weight_input ? nullptr : weights;
-    if (!pb_moe_grouped_supported(width, ff, n_experts) || top <= 0 || top > n_experts) return PB_ERR_BAD_SIZE;
+    if (!pb_moe_grouped_supported(width, ff, n_experts) || n_identity < 0 || top <= 0 || top > n_experts + n_identity) return PB_ERR_BAD_SIZE;
     const int pairs = n * top, tiles = (pairs + kBM - 1) / kBM + n_experts;
     if (tiles > 0x7fffffff / 2 || (ff + kBN - 1) / kBN > 65535 || (width + kBN - 1) / kBN > 65535) return PB_ERR_TOO_LARGE;
     int* offsets = work;
@@ -261,17 +282,17 @@ PB_EXPORT int pb_moe_grouped(const void* h, const void* w_gate_up, const void* w
         // the tcgen05 form: rows gathered into sorted order, then the two grouped products over the same tile list
         int threads = width / 8;
         threads = threads > 256 ? 256 : (threads + 31) / 32 * 32;
-        rc = launch_pdl(moe_gather_rows_kernel, dim3(pairs), dim3(threads), 0, stream, (const bf16*)h, (const int*)sorted, (bf16*)gathered,
-                        width, top);
+        rc = launch_pdl(moe_gather_rows_kernel, dim3(pairs), dim3(threads), 0, stream, (const bf16*)h, (const int*)sorted,
+                        (const int*)(offsets + n_experts), (bf16*)gathered, width, top);
         if (rc != 0) return rc;
-        rc = pb_gemm_tcgen05_grouped(1, PB_BF16, gathered, w_gate_up, act, pairs, 2 * ff, width, n_experts, offsets, tile_expert, tile_row0,
+        rc = pb_gemm_tcgen05_grouped(ungated ? 2 : 1, PB_BF16, gathered, w_gate_up, act, pairs, (ungated ? 1 : 2) * ff, width, n_experts, offsets, tile_expert, tile_row0,
                                      meta, tiles, limit, alpha, shift, sorted, in_weights, stream);
         if (rc != 0) return rc;
         rc = pb_gemm_tcgen05_grouped(0, PB_F32, act, w_down, y, pairs, width, ff, n_experts, offsets, tile_expert, tile_row0, meta, tiles,
                                      0.0f, 1.0f, 0.0f, nullptr, nullptr, stream);
         if (rc != 0) return rc;
         return launch_pdl(moe_combine_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)y, (const int*)place, out_weights,
-                          (const bf16*)add, add_scale, (bf16*)out, width, top, total);
+                          (const bf16*)add, add_scale, (const bf16*)h, (bf16*)out, width, top, total);
     }
     const GatedInter gating(ff, limit > 0.0f ? limit : __builtin_huge_valf(), alpha, shift);
     constexpr int smem0 = kStages * (kBM + 2 * kBN) * kRow * 2, smem1 = kStages * (kBM + kBN) * kRow * 2;
@@ -279,10 +300,15 @@ PB_EXPORT int pb_moe_grouped(const void* h, const void* w_gate_up, const void* w
     if (!configured) {
         cudaError_t ce = cudaFuncSetAttribute(moe_grouped_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem0);
         if (ce == cudaSuccess) ce = cudaFuncSetAttribute(moe_grouped_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1);
+        if (ce == cudaSuccess) ce = cudaFuncSetAttribute(moe_grouped_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1);
         if (ce != cudaSuccess) return (int)ce;
         configured = true;
     }
-    rc = launch_pdl(moe_grouped_kernel<0>, dim3(tiles, (ff + kBN - 1) / kBN), dim3(kThreads), smem0, stream, (const bf16*)h, (const bf16*)w_gate_up,
+    if (ungated)
+        rc = launch_pdl(moe_grouped_kernel<2>, dim3(tiles, (ff + kBN - 1) / kBN), dim3(kThreads), smem1, stream, (const bf16*)h, (const bf16*)w_gate_up,
+                        (const int*)offsets, (const int*)sorted, (const int*)tile_expert, (const int*)tile_row0, (const int*)meta, (bf16*)act,
+                        (float*)nullptr, width, ff, top, gating, (const float*)nullptr);
+    else rc = launch_pdl(moe_grouped_kernel<0>, dim3(tiles, (ff + kBN - 1) / kBN), dim3(kThreads), smem0, stream, (const bf16*)h, (const bf16*)w_gate_up,
                     (const int*)offsets, (const int*)sorted, (const int*)tile_expert, (const int*)tile_row0, (const int*)meta, (bf16*)act,
                     (float*)nullptr, width, ff, top, gating, in_weights);
     if (rc != 0) return rc;
@@ -291,5 +317,5 @@ PB_EXPORT int pb_moe_grouped(const void* h, const void* w_gate_up, const void* w
                     (const int*)meta, (bf16*)nullptr, y, ff, width, top, gating, (const float*)nullptr);
     if (rc != 0) return rc;
     return launch_pdl(moe_combine_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)y, (const int*)place, out_weights,
-                      (const bf16*)add, add_scale, (bf16*)out, width, top, total);
+                      (const bf16*)add, add_scale, (const bf16*)h, (bf16*)out, width, top, total);
 }

@@ -15,7 +15,7 @@
 //                  to 8192 with 16-byte aligned rows, the plain form everything else.  A layer's two ends always take the
 //                  same form, so the fused boundary and the two separate kernels give the same bits.
 //   activation     out = act(in) element by element, in [N, F] float32 or the activation dtype: 0 gelu (erf), 1 gelu (tanh
-//                  form), 2 silu, 3 relu.  float32 arithmetic, one rounding on store.
+//                  form), 2 silu, 3 relu, 4 relu squared.  float32 arithmetic, one rounding on store.
 #include "common.cuh"
 
 #include <stdint.h>
@@ -255,6 +255,7 @@ __device__ __forceinline__ float act_value(float z, int kind) {
     if (kind == 0) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
     if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
     if (kind == 2) return z / (1.0f + expf(-z));
+    if (kind == 4) return squared_relu(z);
     return fmaxf(z, 0.0f);
 }
 
@@ -354,10 +355,10 @@ PB_EXPORT int pb_parallel_add(int dtype, const float* x, const void* a, const vo
     return PB_ERR_BAD_DTYPE;
 }
 
-// in [total] (in_dtype) -> out [total] (out_dtype); kind: 0 gelu (erf), 1 gelu (tanh form), 2 silu, 3 relu.
+// in [total] (in_dtype) -> out [total] (out_dtype); kind: 0 gelu (erf), 1 gelu (tanh form), 2 silu, 3 relu, 4 squared relu.
 PB_EXPORT int pb_activation(int in_dtype, int out_dtype, const void* in, void* out, long long total, int kind, cudaStream_t stream) {
     if (total <= 0) return 0;
-    if (kind < 0 || kind > 3) return PB_ERR_BAD_SIZE;
+    if (kind < 0 || kind > 4) return PB_ERR_BAD_SIZE;
     size_t blocks = ((size_t)total + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     const dim3 grid((unsigned)blocks), block(256);

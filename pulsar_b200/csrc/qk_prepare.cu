@@ -12,6 +12,11 @@
 //                  queries to float32 [N, Hq, D], keys to the key pool (T).  All arithmetic is float32; the pools
 //                  take one rounding.  Hv > 0: Hv value heads of Dv behind the key heads in the row go to the value
 //                  pool as they are.
+//   qk_prepare_whole   the same place where q and k are normed over their whole projections: per token the RMS norm runs over
+//                  all Hq*D query elements (and over all Hkv*D key elements) at once with a weight for each, the heads then
+//                  turn (pairs of neighbours or rotate-half), and the value heads may turn too, over `v_rotary` of their Dv
+//                  dimensions with a table of their own.  One block per (token, section q | k | v), the section's row in
+//                  shared memory.
 //   add_bias       x[n, c] += bias[c] (bias float32): a projection's bias where no kernel behind the product takes it along.
 //   sigmoid_gate_strided   x[n, c] *= sigmoid(gate[n, c / group]) with float32 arithmetic; gate float32 or T, a column slice
 //                  of a wider row; `group` columns of x share a gate column (a gate per head).
@@ -90,6 +95,93 @@ __global__ void qk_prepare_kernel(const TIn* __restrict__ rows, long row_stride,
     }
 }
 
+struct WholeShape {
+    int Hq, Hkv, Hv, D, Dv, rotary, v_rotary, neighbours, page_size;
+    float eps;
+};
+
+template <typename T>
+__device__ __forceinline__ void put(T* dst, size_t at, float v) { dst[at] = from_float<T>(v); }
+
+template <typename TIn, typename T>
+__global__ void qk_prepare_whole_kernel(const TIn* __restrict__ rows, long row_stride, const float* __restrict__ q_norm_w,
+                                        const float* __restrict__ k_norm_w, const float* __restrict__ cos_t,
+                                        const float* __restrict__ sin_t, const float* __restrict__ v_cos, const float* __restrict__ v_sin,
+                                        float* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool,
+                                        const int* __restrict__ slots, const WholeShape sh, const PoolBounds bounds) {
+    pdl_wait();
+    extern __shared__ __align__(16) float x[];           // the section's row
+    __shared__ float scratch[32];
+    const int t = blockIdx.x, section = blockIdx.y;      // 0: queries, 1: keys, 2: values
+    const int heads = section == 0 ? sh.Hq : section == 1 ? sh.Hkv : sh.Hv, D = section == 2 ? sh.Dv : sh.D;
+    const int n = heads * D;
+    const size_t first = section == 0 ? 0 : (size_t)sh.Hq * sh.D + (section == 2 ? (size_t)sh.Hkv * sh.D : 0);
+    int slot = 0;
+    if (section != 0) {
+        slot = slots[t];
+        if (slot < 0 || !slot_ok(slot, sh.page_size, bounds)) return;        // uniform over the block
+    }
+    const TIn* src = rows + (size_t)t * row_stride + first;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = to_float(src[i]); x[i] = v; ss += v * v; }
+    const float* w = section == 0 ? q_norm_w : section == 1 ? k_norm_w : nullptr;
+    float r = 1.0f;
+    if (w != nullptr) r = rsqrtf(block_sum(ss, scratch) / (float)n + sh.eps);
+    __syncthreads();
+    const int rotary = section == 2 ? sh.v_rotary : sh.rotary, turning = rotary >> 1, half = (D + 1) >> 1;
+    const float* c = (section == 2 ? v_cos : cos_t) + (size_t)t * turning;
+    const float* s = (section == 2 ? v_sin : sin_t) + (size_t)t * turning;
+    const size_t page = (size_t)(slot / sh.page_size), in_page = slot % sh.page_size;
+    for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {           // two elements of a head at a time
+        const int head = i / half, j = i - head * half;
+        const bool turns = j < turning;
+        int a, b;                                                            // the pair's places in the head
+        if (sh.neighbours || !turns) { a = 2 * j; b = a + 1; }
+        else { a = j; b = j + turning; }
+        const bool both = b < D;                                             // an odd head's last element stands alone
+        const int ia = head * D + a, ib = head * D + b;
+        float u = x[ia], v = both ? x[ib] : 0.0f;
+        if (w != nullptr) { u = u * r * w[ia]; v = both ? v * r * w[ib] : 0.0f; }
+        if (turns) {
+            const float u0 = u;
+            u = u0 * c[j] - v * s[j];
+            v = v * c[j] + u0 * s[j];
+        }
+        if (section == 0) {
+            const size_t at = (size_t)t * n;
+            q_out[at + ia] = u;
+            if (both) q_out[at + ib] = v;
+        } else {
+            const size_t at = ((page * heads + head) * sh.page_size + in_page) * D;
+            T* dst = section == 1 ? k_pool : v_pool;
+            put(dst, at + a, u);
+            if (both) put(dst, at + b, v);
+        }
+    }
+}
+
+template <typename TIn, typename T>
+int launch_whole(const void* rows, long row_stride, const float* q_norm_w, const float* k_norm_w, const float* cos_t, const float* sin_t,
+                 const float* v_cos, const float* v_sin, float* q_out, void* k_pool, void* v_pool, const int* slots, int n,
+                 const WholeShape& sh, cudaStream_t stream) {
+    int widest = sh.Hq * sh.D;
+    if (sh.Hkv * sh.D > widest) widest = sh.Hkv * sh.D;
+    if (sh.Hv * sh.Dv > widest) widest = sh.Hv * sh.Dv;
+    const size_t smem = sizeof(float) * (size_t)widest;
+    if (smem > 200 * 1024) return PB_ERR_TOO_LARGE;
+    static size_t allowed = 48 * 1024;                     // per instantiation
+    if (smem > allowed) {
+        const cudaError_t e = cudaFuncSetAttribute(qk_prepare_whole_kernel<TIn, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+        allowed = smem;
+    }
+    int threads = 64;
+    while (threads < 512 && threads * 8 < widest) threads <<= 1;
+    return launch_pdl(qk_prepare_whole_kernel<TIn, T>, dim3(n, sh.Hkv > 0 ? 3 : 1), dim3(threads), smem, stream, (const TIn*)rows,
+                      row_stride, q_norm_w, k_norm_w, cos_t, sin_t, v_cos, v_sin, q_out, (T*)k_pool, (T*)v_pool, slots, sh,
+                      pool_bounds_now());
+}
+
 template <typename T, typename TG>
 __global__ void sigmoid_gate_strided_kernel(T* __restrict__ x, const TG* __restrict__ gate, long gate_stride, int width, int group,
                                             size_t total) {
@@ -149,6 +241,32 @@ PB_EXPORT int pb_qk_prepare(int in_dtype, int dtype, const void* rows, long row_
     if (in_dtype == PB_BF16 && dtype == PB_BF16) PB_PREP(__nv_bfloat16, __nv_bfloat16);
     if (in_dtype == PB_BF16 && dtype == PB_F32) PB_PREP(__nv_bfloat16, float);
 #undef PB_PREP
+    return PB_ERR_BAD_DTYPE;
+}
+
+// rows [n, row_stride] of dtype in_dtype: query heads, key heads (D each), value heads (Dv each).  q_norm_w float32 [Hq*D],
+// k_norm_w [Hkv*D] (null: no norm).  cos/sin float32 [n, rotary / 2], v_cos/v_sin [n, v_rotary / 2]; neighbours: elements 2j
+// and 2j + 1 are a pair (else rotate-half).  Queries to q_out float32 [n, Hq, D], keys to k_pool [pages, Hkv, page_size, D], values to
+// v_pool [pages, Hv, page_size, Dv] (dtype).  Hkv 0: the rows hold queries only.
+PB_EXPORT int pb_qk_prepare_whole(int in_dtype, int dtype, const void* rows, long row_stride, const float* q_norm_w, const float* k_norm_w,
+                                  float eps, const float* cos_t, const float* sin_t, const float* v_cos, const float* v_sin,
+                                  float* q_out, void* k_pool, void* v_pool, const int* slots, int n, int Hq, int Hkv, int D, int Hv, int Dv,
+                                  int rotary, int v_rotary, int neighbours, int page_size, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (Hq <= 0 || Hkv < 0 || D <= 0 || rotary < 0 || rotary > D || rotary % 2 || page_size <= 0 || !(eps >= 0.0f) ||
+        (rotary > 0 && (cos_t == nullptr || sin_t == nullptr)))
+        return PB_ERR_BAD_SIZE;
+    if (Hkv > 0 && (Hv <= 0 || Dv <= 0 || v_rotary < 0 || v_rotary > Dv || v_rotary % 2 || k_pool == nullptr ||
+                    v_pool == nullptr || slots == nullptr || (v_rotary > 0 && (v_cos == nullptr || v_sin == nullptr))))
+        return PB_ERR_BAD_SIZE;
+    if (Hkv == 0) Hv = Dv = v_rotary = 0;
+    if (row_stride < (long)(Hq + Hkv) * D + (long)Hv * Dv) return PB_ERR_BAD_SIZE;
+    const WholeShape sh{Hq, Hkv, Hv, D, Dv, rotary, v_rotary, neighbours != 0, page_size, eps};
+#define PB_WHOLE(TI, T) return launch_whole<TI, T>(rows, row_stride, q_norm_w, k_norm_w, cos_t, sin_t, v_cos, v_sin, q_out, k_pool, v_pool, slots, n, sh, stream)
+    if (in_dtype == PB_F32 && dtype == PB_F32) PB_WHOLE(float, float);
+    if (in_dtype == PB_F32 && dtype == PB_BF16) PB_WHOLE(float, __nv_bfloat16);
+    if (in_dtype == PB_BF16 && dtype == PB_BF16) PB_WHOLE(__nv_bfloat16, __nv_bfloat16);
+#undef PB_WHOLE
     return PB_ERR_BAD_DTYPE;
 }
 

@@ -84,15 +84,16 @@ _SIGNATURES = {
     "pb_sample": [_P, _I, _I, _P, _P, _P, _P, _I, _P, _P, _P, _P],
     "pb_sample_workspace": [_I],
     "pb_argmax": [_P, _I, _I, _P, _P, _P],
-    "pb_paged_attention_general": [_I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _P],
+    "pb_paged_attention_general": [_I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _P, _P],
     "pb_attention_general_tiled_supported": [_I, _P, _P, _I, _I, _I, _I, _I, _I],
-    "pb_paged_attention_general_tiled": [_I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _P],
+    "pb_paged_attention_general_tiled": [_I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _P, _P],
     "pb_attention_general_tc_tile": [],
     "pb_attention_general_tc_supported": [_I, _P, _P, _P, _I, _I, _I, _I, _I, _I],
-    "pb_paged_attention_general_tc": [_I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _P],
+    "pb_paged_attention_general_tc": [_I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _P, _P],
     "pb_qkv_split_write": [_I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _P],
     "pb_heads_linear": [_I, _I, _P, _L, _I, _P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _P],
     "pb_latent_prepare": [_I, _P, _L, _P, _L, _P, _F, _P, _P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "pb_latent_norms": [_I, _P, _L, _P, _P, _P, _L, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "pb_latent_expand_keys": [_I, _P, _P, _P, _I, _I, _I, _I, _P],
     "pb_sigmoid_gate": [_I, _P, _P, _L, _I, _I, _P],
     "pb_causal_conv_silu": [_I, _P, _L, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _P],
@@ -106,14 +107,16 @@ _SIGNATURES = {
     "pb_post_norm_add_bias": [_I, _P, _P, _P, _P, _F, _P, _I, _I, _P],
     "pb_glu_bias": [_I, _I, _P, _P, _P, _I, _I, _F, _F, _F, _P],
     "pb_qk_prepare": [_I, _I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _F, _I, _I, _P],
+    "pb_qk_prepare_whole": [_I, _I, _P, _L, _P, _P, _F, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 10 + [_P],
     "pb_sigmoid_gate_strided": [_I, _I, _P, _P, _L, _I, _I, _I, _P],
     "pb_add_bias": [_I, _P, _P, _I, _I, _P],
-    "pb_moe_route": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _I, _F, _P],
+    "pb_moe_route": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _I, _F, _P, _I, _I, _P],
     "pb_moe_gate_up": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _F, _F, _P, _P],
-    "pb_moe_down": [_I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "pb_moe_up": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+    "pb_moe_down": [_I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _I, _P],
     "pb_moe_grouped_workspace": [_I, _I, _I],
     "pb_moe_grouped_supported": [_I, _I, _I],
-    "pb_moe_grouped": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _I, _P, _P],
+    "pb_moe_grouped": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _I, _P, _I, _I, _P],
     "pb_norm_shift": [_I, _P, _P, _F, _P, _P, _L, _P, _P, _P, _P, _P, _P, _I, _I, _P],
     "pb_parallel_add": [_I, _P, _P, _P, _F, _P, _P, _P, _L, _P, _P, _P, _P, _F, _P, _P, _L, _P, _P, _P, _I, _I, _P],
     "pb_activation": [_I, _I, _P, _P, ctypes.c_longlong, _I, _P],
@@ -133,9 +136,9 @@ _LAUNCHERS = {"embed", "scale_cap", "move_ids", "add_rmsnorm", "rope_table", "qk
               "paged_attention_decode_tc_qkv",
               "paged_attention_prefill_tc", "paged_attention_prefill_tcgen05", "gemm_skinny", "gemm_skinny_accumulate",
               "gemm_skinny_scaled", "gemm_tcgen05", "gemm_tcgen05_stream", "gemm_simt", "sample", "argmax", "table_update",
-              "paged_attention_general", "paged_attention_general_tiled", "paged_attention_general_tc", "qkv_split_write", "heads_linear", "latent_prepare", "latent_expand_keys", "sigmoid_gate", "causal_conv_silu",
+              "paged_attention_general", "paged_attention_general_tiled", "paged_attention_general_tc", "qkv_split_write", "heads_linear", "latent_prepare", "latent_norms", "latent_expand_keys", "sigmoid_gate", "causal_conv_silu",
               "selective_scan", "selective_scan_prompt", "selective_scan_chunked", "post_norm_add", "clamped_glu",
-              "post_norm_add_bias", "glu_bias", "qk_prepare", "sigmoid_gate_strided", "add_bias", "moe_route", "moe_gate_up", "moe_down", "moe_grouped",
+              "post_norm_add_bias", "glu_bias", "qk_prepare", "qk_prepare_whole", "sigmoid_gate_strided", "add_bias", "moe_route", "moe_gate_up", "moe_up", "moe_down", "moe_grouped",
               "norm_shift", "parallel_add", "activation", "min_gru", "diff_combine", "retention", "scaled_sum", "concat_streams"}
 
 
@@ -359,16 +362,22 @@ class _Gating:
             fn("pb_set_gating")(0.0, 1.0, 0.0)
 
 
-def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, gating=None) -> bool:
+def _product_mode(swiglu: bool, squared_relu: bool) -> int:
+    assert not (swiglu and squared_relu)
+    return 1 if swiglu else 2 if squared_relu else 0
+
+
+def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, gating=None, squared_relu: bool = False) -> bool:
     """The weight-streaming product for up to 16 tokens (bfloat16).  ``swiglu``: ``w`` holds
     gate rows then up rows and ``out`` [M, inter] receives silu(gate) * up, or with ``gating`` =
     (limit, alpha, shift) the clamped form min(gate, limit) * sigmoid(alpha * .) * (clamp(up) + shift).
+    ``squared_relu``: ``out`` [M, N] receives max(a @ w.T, 0)^2.
     Returns False, having done nothing, when the sizes are not the kernel's."""
     m, k = a.shape
     n = w.shape[0]
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != k:
         return False
-    mode = 1 if swiglu else 0
+    mode = _product_mode(swiglu, squared_relu)
     if not fn("pb_gemm_skinny_supported")(mode, m, n, k):
         return False
     _cuda(a, w, out)
@@ -448,15 +457,15 @@ def linear_prenormed(prepared: torch.Tensor, parts: torch.Tensor, eps: float, w:
     return True
 
 
-def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, gating=None) -> bool:
+def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, gating=None, squared_relu: bool = False) -> bool:
     """The tcgen05 / TMA product for many tokens (bfloat16 operands, float32 accumulation in
-    tensor memory).  ``swiglu`` as in ``gemm_skinny``.  Returns False, having done nothing,
+    tensor memory).  ``swiglu`` and ``squared_relu`` as in ``gemm_skinny``.  Returns False, having done nothing,
     when the sizes are not the kernel's (K must be a multiple of 8)."""
     m, k = a.shape
     n = w.shape[0]
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != k:
         return False
-    mode = 1 if swiglu else 0
+    mode = _product_mode(swiglu, squared_relu)
     if not fn("pb_gemm_tcgen05_supported")(mode, m, n, k):
         return False
     _cuda(a, w, out)
@@ -674,7 +683,7 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
         if out.dtype == torch.bfloat16:
             torch.mm(a, w.t(), out=out)
         else:
-            out.copy_(torch.mm(a, w.t(), out_dtype=torch.float32))
+            torch.mm(a, w.t(), out_dtype=torch.float32, out=out)
 
 
 def gated_linear(ctx, a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, gating=None) -> None:
@@ -938,6 +947,19 @@ def attention(ctx, q: torch.Tensor, cache, out: torch.Tensor, scale: float, wind
                             ctx.seq_of_token, scale, window)
 
 
+def squared_relu_linear(ctx, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """out [M, N] = max(a @ w.T, 0)^2.  In bfloat16, up to 16 rows (the weight-streaming kernel) and more than 128 rows (the
+    tcgen05 kernel) apply it in the product's epilogue; otherwise the product leaves float32 rows for the activation kernel."""
+    if gemm_skinny(a, w, out, squared_relu=True):
+        return
+    fused = GEMM_BACKEND == "tcgen05" or (GEMM_BACKEND == "auto" and a.shape[0] > 128)
+    if fused and gemm_tcgen05(a, w, out, squared_relu=True):
+        return
+    rows = ctx.scratch("mlp.up32", out.shape, torch.float32)
+    linear(a, w, rows)
+    activation(rows, out, "relu2")
+
+
 # ---------------------------------------------------------------- attention in its general form, latent attention
 # The general attention has two kernels: the tiled one (keys and values of a tile staged in shared memory and shared by 16
 # query rows; splits of the keys where the rows alone do not fill the GPU) for rows that are multiples of 16 bytes, and the
@@ -969,7 +991,8 @@ def paged_attention_general(ctx, q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                             slopes: Optional[torch.Tensor] = None, key_width: Optional[int] = None,
                             value_width: Optional[int] = None, tiled: Optional[bool] = None,
                             tensor_cores: Optional[bool] = None, keep_first: int = 0, softcap: Optional[float] = None,
-                            sinks: Optional[torch.Tensor] = None, v_share: int = 1) -> None:
+                            sinks: Optional[torch.Tensor] = None, v_share: int = 1, sigmoid: bool = False,
+                            score_bias: Optional[torch.Tensor] = None, turn_back=None) -> None:
     """Attention of the step's tokens (``ctx``: cu_q, kv_len, seq_of_token, host.q_lens) with float32 queries ``q``
     [N, Hq, Dk] over pools [pages, Hkv, page, stride]: keys are the first ``key_width`` (default: all) elements of a
     ``k_pool`` row, values the first ``value_width`` of a ``v_pool`` row (the two may be one tensor).  ``slopes`` [Hq]
@@ -980,8 +1003,11 @@ def paged_attention_general(ctx, q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
     tensor-core kernel for steps with portions where it applies, False never, True insists.
     ``v_share``: that many consecutive key heads read one value head (``v_pool`` has Hkv / v_share heads): several score
     maps over the same values.  ``out`` has the pools' dtype or float32 (rows that are subtracted from one another afterwards
-    stay unrounded)."""
-    _cuda(q, k_pool, v_pool, out, block_table, slopes, sinks)
+    stay unrounded).
+    ``sigmoid``: a visible key's weight is sigmoid(score + score_bias[h]) (``score_bias`` [Hq] float32 or None) and the weights
+    are not normalised.  ``turn_back`` = (cos, sin), float32 [N, Dv / 2]: a token's output row turns back by its angles, columns
+    2m and 2m + 1 a pair, before it is rounded (for values that were cached turned by their own positions)."""
+    _cuda(q, k_pool, v_pool, out, block_table, slopes, sinks, score_bias)
     _check_against(k_pool)
     n, hq, dk = q.shape
     keep_first, softcap = int(keep_first or 0), float(softcap or 0.0)
@@ -997,6 +1023,14 @@ def paged_attention_general(ctx, q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
     assert v_pool.shape[:3] == (pages, hkv // v_share, page_size)
     assert block_table.dtype == torch.int32 and block_table.dim() == 2
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == hq)
+    assert score_bias is None or (sigmoid and score_bias.dtype == torch.float32 and score_bias.numel() == hq)
+    assert not (sigmoid and sinks is not None)
+    out_cos = out_sin = None
+    if turn_back is not None:
+        out_cos, out_sin = turn_back
+        _cuda(out_cos, out_sin)
+        assert out_cos.dtype == out_sin.dtype == torch.float32 and out_cos.shape == out_sin.shape == (n, dv // 2) and dv % 2 == 0
+    weighting = (1 if sigmoid else 0, _p(score_bias), _p(out_cos), _p(out_sin))
     q_lens = ctx.host.q_lens
     insist = tensor_cores is True
     if tensor_cores is None:
@@ -1010,7 +1044,7 @@ def paged_attention_general(ctx, q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
             check(fn("pb_paged_attention_general_tc")(pool_code, _p(q), _p(k_pool), _p(v_pool), _p(out), _p(block_table),
                                                       block_table.shape[1], _p(ctx.cu_q), _p(ctx.kv_len), _p(slopes), len(q_lens),
                                                       n_q_tiles, hq, hkv, dk, dv, k_stride, v_stride, page_size, float(scale),
-                                                      int(window or 0), int(chunk or 0), keep_first, softcap, _p(sinks), v_share, out_f32, stream()),
+                                                      int(window or 0), int(chunk or 0), keep_first, softcap, _p(sinks), v_share, out_f32, *weighting, stream()),
                   "paged_attention_general_tc")
             return
         if insist:
@@ -1027,13 +1061,13 @@ def paged_attention_general(ctx, q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                                                      _p(block_table), block_table.shape[1], _p(ctx.cu_q), _p(ctx.kv_len),
                                                      _p(slopes), n, len(ctx.host.q_lens), row_tiles, n_splits, hq, hkv, dk, dv,
                                                      k_stride, v_stride, page_size, float(scale), int(window or 0),
-                                                     int(chunk or 0), keep_first, softcap, _p(sinks), v_share, out_f32, stream()),
+                                                     int(chunk or 0), keep_first, softcap, _p(sinks), v_share, out_f32, *weighting, stream()),
               "paged_attention_general_tiled", kernels=2 if n_splits > 1 else 1)
         return
     check(fn("pb_paged_attention_general")(pool_code, _p(q), _p(k_pool), _p(v_pool), _p(out), _p(block_table),
                                            block_table.shape[1], _p(ctx.cu_q), _p(ctx.kv_len), _p(ctx.seq_of_token), _p(slopes),
                                            n, hq, hkv, dk, dv, k_stride, v_stride, page_size, float(scale), int(window or 0),
-                                           int(chunk or 0), keep_first, softcap, _p(sinks), v_share, out_f32, stream()), "paged_attention_general")
+                                           int(chunk or 0), keep_first, softcap, _p(sinks), v_share, out_f32, *weighting, stream()), "paged_attention_general")
 
 
 def qkv_split_write(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
@@ -1108,6 +1142,33 @@ def latent_prepare(q: torch.Tensor, down: Optional[torch.Tensor], norm_weight: O
                                   _p(sin), _p(slots), _p(pool), _p(q_out), front + rot_dim, front, 1 if plain_too else 0,
                                   _p(latent_out), _p(rot_out), n, n_heads, dim, rot_dim, rot_dims, rank, page_size, stream()),
           "latent_prepare")
+
+
+def latent_norms(q_lat: torch.Tensor, q_norm: torch.Tensor, q_out: torch.Tensor, eps: float, down: Optional[torch.Tensor],
+                 norm_weight: Optional[torch.Tensor], cos: torch.Tensor, sin: torch.Tensor, slots: Optional[torch.Tensor],
+                 pool: Optional[torch.Tensor], rank: int, rot_dim: int, page_size: int, latent_out: Optional[torch.Tensor] = None,
+                 rot_out: Optional[torch.Tensor] = None) -> None:
+    """q_out [N, q_rank] = rmsnorm(q_lat) * q_norm (the queries' latent, ready for its expansion), and where ``down`` is given what
+    ``latent_prepare`` does with it.  ``q_lat`` and ``down`` may be column slices of one tensor."""
+    _cuda(q_norm, q_out, norm_weight, cos, sin, slots, pool, latent_out, rot_out)
+    n, q_rank = q_lat.shape
+    assert q_lat.is_cuda and q_lat.stride(1) == 1 and q_out.shape == (n, q_rank) and q_out.dtype == q_lat.dtype
+    assert q_norm.dtype == torch.float32 and q_norm.numel() == q_rank
+    assert cos.dtype == torch.float32 and cos.shape == sin.shape and cos.shape[0] == n
+    down_tok = 0
+    if down is not None:
+        assert down.dtype == q_lat.dtype and down.shape == (n, rank + rot_dim) and down.stride(1) == 1
+        assert norm_weight.dtype == torch.float32 and norm_weight.numel() == rank and slots.dtype == torch.int32
+        assert pool.dtype == q_lat.dtype and pool.shape[1:] == (1, page_size, rank + rot_dim)
+        _check_against(pool)
+        down_tok = down.stride(0)
+        for t, width in ((latent_out, rank), (rot_out, rot_dim)):
+            assert t is None or (t.dtype == q_lat.dtype and t.shape == (n, width))
+    else:
+        assert latent_out is None and rot_out is None
+    check(fn("pb_latent_norms")(code(q_lat.dtype), _p(q_lat), q_lat.stride(0), _p(q_norm), _p(q_out), _p(down), down_tok, _p(norm_weight),
+                                float(eps), _p(cos), _p(sin), _p(slots), _p(pool), _p(latent_out), _p(rot_out), n, q_rank, rank, rot_dim,
+                                2 * cos.shape[1], page_size, stream()), "latent_norms")
 
 
 def latent_expand_keys(plain: torch.Tensor, shared: torch.Tensor, keys: torch.Tensor) -> None:
@@ -1286,6 +1347,40 @@ def qk_prepare(rows: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[torch.T
                               int(n_value_heads), int(value_dim), stream()), "qk_prepare")
 
 
+def qk_prepare_whole(rows: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
+                     slots: Optional[torch.Tensor], n_heads: int, n_kv_heads: int, head_dim: int, value_dim: int, page_size: int,
+                     q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float, turn=None, v_turn=None,
+                     neighbours: bool = True) -> None:
+    """Split the projection rows [q: Hq*D | k: Hkv*D | v: Hkv*Dv] (float32 or the pools' dtype) with q and k normed over their
+    whole projections (``q_norm`` float32 [Hq*D], ``k_norm`` [Hkv*D]; None: no norm), then turned by ``turn`` = (cos, sin) (float32
+    [N, rotary / 2], pairs of neighbours or rotate-half over a head's first ``rotary`` dimensions), the values turned by ``v_turn``
+    over theirs.  Queries to float32 ``q_out`` [N, Hq, D], keys and values into their pages.  ``n_kv_heads`` 0: queries only."""
+    _cuda(q_out, k_pool, v_pool, slots, q_norm, k_norm)
+    _check_against(k_pool)
+    n = rows.shape[0]
+    assert rows.is_cuda and rows.stride(1) == 1 and rows.shape[1] >= (n_heads + n_kv_heads) * head_dim + n_kv_heads * value_dim
+    assert q_out.dtype == torch.float32 and q_out.shape == (n, n_heads, head_dim)
+    assert q_norm is None or (q_norm.dtype == torch.float32 and q_norm.numel() == n_heads * head_dim)
+    pool_dtype = rows.dtype
+    if n_kv_heads:
+        assert k_norm is None or (k_norm.dtype == torch.float32 and k_norm.numel() == n_kv_heads * head_dim)
+        assert slots.dtype == torch.int32 and k_pool.shape[1:] == (n_kv_heads, page_size, head_dim) and v_pool.dtype == k_pool.dtype
+        assert v_pool.shape[1:] == (n_kv_heads, page_size, value_dim)
+        pool_dtype = k_pool.dtype
+    tables = []
+    for pair, width in ((turn, head_dim), (v_turn if n_kv_heads else None, value_dim)):
+        cos, sin = pair if pair is not None else (None, None)
+        if pair is not None:
+            _cuda(cos, sin)
+            assert cos.dtype == sin.dtype == torch.float32 and cos.shape == sin.shape and cos.shape[0] == n and 2 * cos.shape[1] <= width
+        tables.append((cos, sin, 0 if pair is None else 2 * cos.shape[1]))
+    (cos, sin, rotary), (v_cos, v_sin, v_rotary) = tables
+    check(fn("pb_qk_prepare_whole")(code(rows.dtype), code(pool_dtype), _p(rows), rows.stride(0), _p(q_norm), _p(k_norm) if n_kv_heads else None,
+                                    float(eps), _p(cos), _p(sin), _p(v_cos), _p(v_sin), _p(q_out), _p(k_pool), _p(v_pool), _p(slots), n,
+                                    n_heads, n_kv_heads, head_dim, n_kv_heads, value_dim, rotary, v_rotary, 1 if neighbours else 0,
+                                    page_size, stream()), "qk_prepare_whole")
+
+
 def sigmoid_gate_strided(x: torch.Tensor, gate: torch.Tensor, group: int = 1) -> None:
     """x[n, c] *= sigmoid(gate[n, c // group]) in place (float32 arithmetic); ``gate`` float32 or of x's dtype, possibly a column
     slice.  ``group`` neighbouring columns of x share one gate column (a head's width: one gate per head)."""
@@ -1306,13 +1401,16 @@ def add_bias(x: torch.Tensor, bias: torch.Tensor) -> None:
 
 # ---------------------------------------------------------------- mixture of experts
 def moe_route(h: torch.Tensor, router: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, scale: float = 1.0,
-              renormalize: bool = False, extra: Optional[torch.Tensor] = None, softmax: bool = False, renorm_eps: float = 0.0) -> None:
+              renormalize: bool = False, extra: Optional[torch.Tensor] = None, softmax: bool = False, renorm_eps: float = 0.0,
+              correction: Optional[torch.Tensor] = None, groups: Optional[Tuple[int, int]] = None) -> None:
     """ids [N, top] int32 and weights [N, top] float32 of the ``top`` largest sigmoid(router @ h) per token (float32 sums;
     ties go to the lower index), weights times ``scale`` (after division by their sum with ``renormalize``).  With ``extra``
     (float32 [N, X]) the router has X more rows behind the experts' that compete for nothing: their sigmoids go there.
     ``softmax``: the scores are softmax(router @ h) over all experts instead; ``renorm_eps`` is added to the chosen scores' sum
-    before the division."""
-    _cuda(h, router, ids, weights, extra)
+    before the division.  ``correction`` (float32 [E]): the choice goes by score + correction, the weights by the score alone.
+    ``groups`` = (count, keep): the experts form ``count`` groups of neighbours, a group counts as its best choice score, and
+    only experts of the ``keep`` best groups can be chosen."""
+    _cuda(h, router, ids, weights, extra, correction)
     n, width = h.shape
     n_extra = 0 if extra is None else extra.shape[1]
     e = router.shape[0] - n_extra
@@ -1320,8 +1418,11 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, ids: torch.Tensor, weights:
     assert router.dtype == torch.float32 and router.shape == (e + n_extra, width) and ids.dtype == torch.int32 and ids.shape == (n, top)
     assert weights.dtype == torch.float32 and weights.shape == (n, top)
     assert extra is None or (extra.dtype == torch.float32 and extra.shape == (n, n_extra))
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == e)
+    n_groups, keep = (1, 1) if groups is None else (int(groups[0]), int(groups[1]))
     check(fn("pb_moe_route")(code(h.dtype), _p(h), _p(router), _p(ids), _p(weights), n, width, e, top, float(scale),
-                             1 if renormalize else 0, n_extra, _p(extra), 1 if softmax else 0, float(renorm_eps), stream()), "moe_route")
+                             1 if renormalize else 0, n_extra, _p(extra), 1 if softmax else 0, float(renorm_eps), _p(correction), n_groups,
+                             keep, stream()), "moe_route")
 
 
 def moe_gate_up(h: torch.Tensor, w_gate_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor, gating,
@@ -1341,11 +1442,25 @@ def moe_gate_up(h: torch.Tensor, w_gate_up: torch.Tensor, ids: torch.Tensor, act
                                float(alpha), float(shift), _p(in_weights), stream()), "moe_gate_up")
 
 
+def moe_up(h: torch.Tensor, w_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor) -> None:
+    """act [N * top, ff] = max(w_up[e] @ h, 0)^2 of every token's chosen experts (ungated experts; ``w_up`` [E, ff, width]);
+    rows of pairs with ids >= E (identity experts) are left as they are."""
+    _cuda(h, w_up, ids, act)
+    n, width = h.shape
+    e, ff, w2 = w_up.shape
+    top = ids.shape[1]
+    assert w2 == width and act.shape == (n * top, ff) and h.dtype == w_up.dtype == act.dtype
+    assert ids.dtype == torch.int32 and ids.shape[0] == n
+    check(fn("pb_moe_up")(code(h.dtype), _p(h), _p(w_up), _p(ids), _p(act), n, width, ff, top, e, stream()), "moe_up")
+
+
 def moe_down(act: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: Optional[torch.Tensor], add: Optional[torch.Tensor],
-             out: torch.Tensor, add_scale: Optional[torch.Tensor] = None) -> None:
+             out: torch.Tensor, add_scale: Optional[torch.Tensor] = None, identity: Optional[torch.Tensor] = None) -> None:
     """out [N, width] = add * add_scale + sum over a token's chosen experts, in the order of ``ids``, of weight * (w_down[e] @
-    act row).  ``weights`` None: every pair counts once; ``add_scale`` (float32 [N]) None: 1."""
-    _cuda(act, w_down, ids, weights, add, out, add_scale)
+    act row).  ``weights`` None: every pair counts once; ``add_scale`` (float32 [N]) None: 1.  ``identity`` [N, width]: what a pair
+    with an id >= E contributes (times its weight) in place of an expert's output."""
+    _cuda(act, w_down, ids, weights, add, out, add_scale, identity)
+    assert identity is None or (identity.shape == out.shape and identity.dtype == out.dtype)
     n, width = out.shape
     e, w2, ff = w_down.shape
     top = ids.shape[1]
@@ -1355,7 +1470,7 @@ def moe_down(act: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights
     assert add is None or (add.shape == out.shape and add.dtype == out.dtype)
     assert add_scale is None or (add_scale.dtype == torch.float32 and add_scale.numel() == n)
     check(fn("pb_moe_down")(code(out.dtype), _p(act), _p(w_down), _p(ids), _p(weights), _p(add), _p(add_scale), _p(out), n, width, ff,
-                            top, stream()), "moe_down")
+                            top, _p(identity), e, stream()), "moe_down")
 
 
 # Steps of more than MOE_GROUPED_MIN tokens (bfloat16) sort their (token, expert) pairs by expert on the device and run every
@@ -1383,19 +1498,20 @@ def moe_grouped_workspace(n: int, top: int, n_experts: int) -> int:
 def moe_grouped(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                 add: Optional[torch.Tensor], act: torch.Tensor, y: torch.Tensor, out: torch.Tensor, work: torch.Tensor, gating,
                 gathered: Optional[torch.Tensor] = None, weight_input: bool = False,
-                add_scale: Optional[torch.Tensor] = None) -> None:
+                add_scale: Optional[torch.Tensor] = None, ungated: bool = False, identity: int = 0) -> None:
     """What ``moe_gate_up`` and ``moe_down`` compute together, for steps of many tokens (bfloat16): pairs sorted by expert, the
     experts' products in tensor-core tiles, the weighted sum in the order of ``ids``.  ``act`` [N * top, ff] bfloat16, ``y``
     [N * top, width] float32 and ``work`` (int32, ``moe_grouped_workspace`` elements) are scratch.  With ``gathered``
     (bfloat16 [N * top, width] scratch) the products run on the grouped tcgen05 kernel, else on mma.sync.  ``weight_input``: a
     pair's weight multiplies its expert's input (inside the gate/up epilogue) instead of its output; ``add_scale`` (float32
-    [N]) multiplies ``add``."""
+    [N]) multiplies ``add``.  ``ungated``: ``w_gate_up`` is [E, ff, width] and an expert's unit is max(w_up h, 0)^2 (``moe_up``).
+    ``identity``: that many ids behind the experts' stand for the token's own row of ``h``."""
     _cuda(h, w_gate_up, w_down, ids, weights, add, act, y, out, work, gathered, add_scale)
     assert add_scale is None or (add_scale.dtype == torch.float32 and add_scale.numel() == h.shape[0])
     assert gathered is None or (gathered.dtype == torch.bfloat16 and gathered.shape == (h.shape[0] * ids.shape[1], h.shape[1]))
     n, width = h.shape
     e, two_ff, w2 = w_gate_up.shape
-    ff, top = two_ff // 2, ids.shape[1]
+    ff, top = two_ff if ungated else two_ff // 2, ids.shape[1]
     assert h.dtype == w_gate_up.dtype == w_down.dtype == act.dtype == out.dtype == torch.bfloat16 and w2 == width
     assert w_down.shape == (e, width, ff) and ids.dtype == torch.int32 and ids.shape == weights.shape == (n, top)
     assert weights.dtype == torch.float32 and act.shape == (n * top, ff) and y.dtype == torch.float32 and y.shape == (n * top, width)
@@ -1404,7 +1520,7 @@ def moe_grouped(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     limit, alpha, shift = gating if gating is not None else (0.0, 1.0, 0.0)
     check(fn("pb_moe_grouped")(_p(h), _p(w_gate_up), _p(w_down), _p(ids), _p(weights), _p(add), _p(act), _p(y), _p(out), _p(work),
                                _p(gathered), n, width, ff, e, top, float(limit), float(alpha), float(shift), 1 if weight_input else 0,
-                               _p(add_scale), stream()), "moe_grouped",
+                               _p(add_scale), 1 if ungated else 0, int(identity), stream()), "moe_grouped",
           kernels=4 if gathered is None else 5)
 
 
@@ -1454,12 +1570,12 @@ def parallel_add(ctx, residual: torch.Tensor, a: torch.Tensor, b: Optional[torch
                                 stream()), "parallel_add")
 
 
-ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2, "relu": 3}
+ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "relu2": 4}
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> None:
     """out = act(x) element by element in float32, one rounding on store; ``kind``: "gelu" (the erf form), "gelu_tanh",
-    "silu", "relu".  ``x`` float32 or of ``out``'s dtype."""
+    "silu", "relu", "relu2" (max(x, 0)^2).  ``x`` float32 or of ``out``'s dtype."""
     _cuda(x, out)
     assert x.shape == out.shape and kind in ACTIVATIONS
     check(fn("pb_activation")(code(x.dtype), code(out.dtype), _p(x), _p(out), x.numel(), ACTIVATIONS[kind], stream()), "activation")

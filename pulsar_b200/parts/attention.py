@@ -48,6 +48,12 @@ class Attention(Mixer):
     exp(<lq2, lk2>) + d.  ``spec.q_temperature`` = (coef, every) multiplies the query at position p by
     1 + coef * ln(floor((p + 1) / every) + 1) (float32, as the queries are split off the projection row).
 
+    Further members of the general form: with ``qk_norm_whole`` q and k are normed over their whole projections (one weighted
+    norm for all query heads together, one for all key heads) before the rotation, with ``rotate_neighbours`` the rotation
+    pairs elements 2i and 2i + 1, and with ``value_position`` the values turn by their positions before they are cached and
+    every head's output turns back by the query's, inside the attention kernels (``ops.qk_prepare_whole``, ``turn_back``).
+    ``sigmoid_weights``: the weight of a visible key is sigmoid(score + score_bias[head]) and nothing is normalised.
+
     ``output_bias`` is the output projection's bias (or None).  ``forward`` adds it unless the block has set
     ``defer_output_bias`` because the kernel behind the mixer takes it along.
     """
@@ -62,17 +68,32 @@ class Attention(Mixer):
         # q | k, so the gate's columns ride along in the same product)
         self.prepared = bool(spec.bias or spec.values_from_keys or not spec.qk_norm_weight or spec.qk_norm_after_rotation
                              or spec.output_gate)
+        # what only ops.qk_prepare_whole does
+        self.whole = bool(spec.qk_norm_whole or spec.rotate_neighbours or spec.value_position is not None)
+        if self.whole and (self.prepared or spec.differential is not None or spec.q_temperature is not None or not spec.own_kv):
+            raise ValueError("attention: the norm over whole projections, the neighbours' rotation and turned values go with plain "
+                             "projections of its own keys and values")
+        if spec.qk_norm_whole and spec.qk_norm_eps is None:
+            raise ValueError("attention: the norm over whole projections needs its eps")
+        if self.whole and spec.qk_norm_eps is not None and not spec.qk_norm_whole:
+            raise ValueError("attention: the neighbours' rotation and turned values have no per-head norm beside them")
+        if spec.value_position is not None and spec.value_position.rotary_dim != spec.value_dim:
+            raise ValueError("attention: values turn over all their dimensions")
+        if spec.score_bias and not spec.sigmoid_weights:
+            raise ValueError("attention: a score bias per head goes with sigmoid weights (a softmax does not see it)")
+        if spec.sigmoid_weights and (spec.sinks or spec.fixed_sink is not None):
+            raise ValueError("attention: sigmoid weights have no denominator that a sink could join")
         self.maps = 2 if spec.differential is not None else 1          # score maps per head
         self.general = bool(spec.value_dim != spec.head_dim or spec.chunk is not None or spec.distance_bias is not None
                             or spec.keep_first or spec.softcap is not None or spec.sinks or spec.fixed_sink is not None
-                            or spec.output_gate or self.prepared
+                            or spec.output_gate or self.prepared or self.whole or spec.sigmoid_weights
                             or self.maps > 1 or spec.q_temperature is not None)
         if (self.maps > 1 or spec.q_temperature is not None) and (self.prepared or not spec.own_kv):
             raise ValueError("attention: the differential form and the query temperature go with plain projections of its own keys")
         if spec.q_temperature is not None and not (int(spec.q_temperature[1]) > 0):
             raise ValueError("attention: the query temperature's period must be positive")
         if self.general:
-            if not self.prepared and (spec.position is not None or spec.qk_norm_eps is not None):
+            if not self.prepared and not self.whole and (spec.position is not None or spec.qk_norm_eps is not None):
                 raise ValueError("attention: the general form (value width, chunk mask, distance bias) has neither rotation nor q/k norm")
             if self.prepared:
                 if spec.qk_norm_eps is not None and spec.qk_norm_weight == spec.qk_norm_after_rotation:
@@ -91,6 +112,10 @@ class Attention(Mixer):
             raise ValueError("attention: window must be positive")
         self.spec, self.prefix, self.dtype = spec, prefix, dtype
         self.position = POSITIONS.get(spec.position.kind)(spec.position) if spec.position is not None else None
+        self.value_position = None
+        if spec.value_position is not None:
+            self.value_position = POSITIONS.get(spec.value_position.kind)(spec.value_position)
+        self.score_bias = None
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.slopes = None
         self.q_bias = self.k_bias = self.sinks = None
         name = spec.tensor_name
@@ -98,7 +123,7 @@ class Attention(Mixer):
                       "o": name("o", "o_proj.weight"), "q_norm": name("q_norm", "q_norm.weight"),
                       "k_norm": name("k_norm", "k_norm.weight"), "gate": name("gate", "g_proj.weight"),
                       "sinks": name("sinks", "sinks"), "lq1": name("lq1", "lambda_q1"), "lk1": name("lk1", "lambda_k1"),
-                      "lq2": name("lq2", "lambda_q2"), "lk2": name("lk2", "lambda_k2")}
+                      "lq2": name("lq2", "lambda_q2"), "lk2": name("lk2", "lambda_k2"), "score_bias": name("score_bias", "score_bias")}
         self.diff_lambda = 0.0
         for role in ("q", "k", "o"):          # a bias is named after its weight unless the specification names it
             weight = self.names[role]
@@ -124,12 +149,15 @@ class Attention(Mixer):
             specs.append(WeightSpec(p + nm["o_bias"], (s.hidden,), role="vector", init="small"))
         if s.sinks:
             specs.append(WeightSpec(p + nm["sinks"], (s.n_heads,), role="vector", init="small"))
+        if s.score_bias:
+            specs.append(WeightSpec(p + nm["score_bias"], (s.n_heads,), role="vector", init="small"))
         if self.maps > 1:
             specs += [WeightSpec(p + nm[r], (s.head_dim,), role="vector", init="small") for r in ("lq1", "lk1", "lq2", "lk2")]
         if s.qk_norm_eps is not None and s.qk_norm_weight:
-            specs.append(WeightSpec(p + nm["q_norm"], (s.head_dim,), role="vector", init="ones_normal"))
+            q_heads, k_heads = (s.n_heads, s.n_kv_heads) if s.qk_norm_whole else (1, 1)
+            specs.append(WeightSpec(p + nm["q_norm"], (q_heads * s.head_dim,), role="vector", init="ones_normal"))
             if s.own_kv:
-                specs.append(WeightSpec(p + nm["k_norm"], (s.head_dim,), role="vector", init="ones_normal"))
+                specs.append(WeightSpec(p + nm["k_norm"], (k_heads * s.head_dim,), role="vector", init="ones_normal"))
         return specs
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -159,6 +187,8 @@ class Attention(Mixer):
             self.sinks = tensors[p + nm["sinks"]]
         elif s.fixed_sink is not None:
             self.sinks = torch.full((s.n_heads,), float(s.fixed_sink), dtype=torch.float32, device=self.w_o.device)
+        if s.score_bias:
+            self.score_bias = tensors[p + nm["score_bias"]]
         if s.qk_norm_eps is not None and s.qk_norm_weight:
             self.q_norm = tensors[p + nm["q_norm"]]
             self.k_norm = tensors.get(p + nm["k_norm"])
@@ -167,7 +197,8 @@ class Attention(Mixer):
             self.slopes = torch.tensor(slopes, dtype=torch.float64).to(torch.float32).to(self.w_o.device)
 
     def weight_bytes(self) -> int:
-        ts = [self.w_qkv, self.w_o, self.q_norm, self.k_norm, self.slopes, self.q_bias, self.k_bias, self.output_bias, self.sinks]
+        ts = [self.w_qkv, self.w_o, self.q_norm, self.k_norm, self.slopes, self.q_bias, self.k_bias, self.output_bias, self.sinks,
+              self.score_bias]
         return sum(t.numel() * t.element_size() for t in ts if t is not None)
 
     def cache_need(self) -> CacheNeed:
@@ -205,7 +236,13 @@ class Attention(Mixer):
         n_kv = s.n_kv_heads if s.own_kv else 0
         maps = self.maps
         q = ctx.scratch("attn.q32", (n, s.n_heads * maps, s.head_dim), torch.float32)
-        if self.prepared:
+        turn_back = None
+        if self.whole:
+            turn = self.position.tables(ctx) if self.position is not None else None
+            turn_back = self.value_position.tables(ctx) if self.value_position is not None else None
+            ops.qk_prepare_whole(qkv, q, cache.k_pool, cache.v_pool, cache.slots, s.n_heads, n_kv, s.head_dim, s.value_dim, cache.page_size,
+                                 self.q_norm, self.k_norm, s.qk_norm_eps or 0.0, turn, turn_back, s.rotate_neighbours)
+        elif self.prepared:
             cos = sin = None
             rotary = 0
             if self.position is not None:
@@ -229,7 +266,8 @@ class Attention(Mixer):
         else:
             o = ctx.scratch("attn.o", (n, s.n_heads * maps, s.value_dim))
         ops.paged_attention_general(ctx, q, cache.k_pool, cache.v_pool, o, cache.block_table, s.scale, s.window, s.chunk,
-                                    self.slopes, keep_first=s.keep_first, softcap=s.softcap, sinks=self.sinks, v_share=maps)
+                                    self.slopes, keep_first=s.keep_first, softcap=s.softcap, sinks=self.sinks, v_share=maps,
+                                    sigmoid=s.sigmoid_weights, score_bias=self.score_bias, turn_back=turn_back)
         if maps > 1:
             both, o = o, ctx.scratch("attn.o.diff", (n, s.n_heads, s.value_dim))
             ops.diff_combine(both, o, s.n_kv_heads, self.diff_lambda, s.norm_eps, 1.0 - float(s.differential))

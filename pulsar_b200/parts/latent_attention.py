@@ -36,12 +36,16 @@ class LatentAttention(Mixer):
     exponential joins the softmax's denominator (tensor role "sinks").  ``spec.position`` gives the rotation (its table's
     ``rotary_dim`` leading dimensions of the rotated part turn, in neighbouring pairs).  With ``own_kv`` False the
     mixer has no down projection and attends over the rows another layer cached this step, with its own expansions.
+    With ``q_rank`` the queries come out of a latent of their own: a down projection of the input (role "q_down") gives
+    ``q_rank`` numbers, RMS-normed with ``latent_norm_eps`` and a weight (role "q_norm"), which the query projection (role "q")
+    expands.  The two down projections are one product, the two norms one kernel (``ops.latent_norms``).
     """
 
     def __init__(self, spec: MixerSpec, prefix: str, dtype: torch.dtype):
         self.rank = int(spec.option("kv_rank", 0))
         self.rot_dim = int(spec.option("rot_dim", 0))
         self.norm_eps = float(spec.option("latent_norm_eps", 1e-6))
+        self.q_rank = int(spec.option("q_rank", 0) or 0)
         self.gated = bool(spec.option("gated", False))
         self.head_gate = bool(spec.option("head_gate", False))
         if self.gated and self.head_gate:
@@ -58,8 +62,10 @@ class LatentAttention(Mixer):
         self.names = {r: name(r, d) for r, d in (("q", "q_proj.weight"), ("down", "kv_down_proj.weight"),
                                                  ("latent_norm", "kv_norm.weight"), ("up_k", "k_up_proj.weight"),
                                                  ("up_v", "v_up_proj.weight"), ("gate", "gate_proj.weight"),
-                                                 ("o", "o_proj.weight"), ("sinks", "sinks"))}
+                                                 ("o", "o_proj.weight"), ("sinks", "sinks"),
+                                                 ("q_down", "q_down_proj.weight"), ("q_norm", "q_norm.weight"))}
         self.sinks = None
+        self.w_q = self.q_norm = None
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.latent_norm = self.w_uk_rows = self.w_uv_rows = None
 
     @property
@@ -69,7 +75,11 @@ class LatentAttention(Mixer):
     # ---------------------------------------------------------------- weights
     def weight_specs(self) -> List[WeightSpec]:
         s, p, nm = self.spec, self.prefix, self.names
-        specs = [WeightSpec(p + nm["q"], (s.n_heads * (s.head_dim + self.rot_dim), s.hidden))]
+        specs = []
+        if self.q_rank:
+            specs += [WeightSpec(p + nm["q_down"], (self.q_rank, s.hidden)),
+                      WeightSpec(p + nm["q_norm"], (self.q_rank,), role="vector", init="ones_normal")]
+        specs.append(WeightSpec(p + nm["q"], (s.n_heads * (s.head_dim + self.rot_dim), self.q_rank or s.hidden)))
         if s.own_kv:
             specs += [WeightSpec(p + nm["down"], (self.row, s.hidden)),
                       WeightSpec(p + nm["latent_norm"], (self.rank,), role="vector", init="ones_normal")]
@@ -84,7 +94,9 @@ class LatentAttention(Mixer):
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         s, p, nm = self.spec, self.prefix, self.names
-        rows = [tensors[p + nm["q"]]]
+        rows = [tensors[p + nm["q_down" if self.q_rank else "q"]]]
+        if self.q_rank:
+            self.w_q, self.q_norm = tensors[p + nm["q"]], tensors[p + nm["q_norm"]]
         if s.own_kv:
             rows.append(tensors[p + nm["down"]])
             self.latent_norm = tensors[p + nm["latent_norm"]]
@@ -92,7 +104,7 @@ class LatentAttention(Mixer):
             rows.append(tensors[p + nm["gate"]])
         if s.sinks:
             self.sinks = tensors[p + nm["sinks"]]
-        self.w_in = torch.cat(rows, dim=0).contiguous() if len(rows) > 1 else rows[0]      # rows: q | down | gate
+        self.w_in = torch.cat(rows, dim=0).contiguous() if len(rows) > 1 else rows[0]      # rows: q (or its latent) | down | gate
         # per head [inputs, outputs]: the key expansion as stored serves the query side (head_dim -> rank), the value
         # expansion is transposed once (rank -> value_dim)
         self.w_uk_t = tensors[p + nm["up_k"]].view(s.n_heads, s.head_dim, self.rank).contiguous()
@@ -101,7 +113,7 @@ class LatentAttention(Mixer):
         self.w_o = tensors[p + nm["o"]]
 
     def weight_bytes(self) -> int:
-        ts = [self.w_in, self.w_uk_t, self.w_uv, self.w_o, self.latent_norm, self.sinks]      # a step reads one form of the expansions
+        ts = [self.w_in, self.w_q, self.q_norm, self.w_uk_t, self.w_uv, self.w_o, self.latent_norm, self.sinks]      # a step reads one form of the expansions
         return sum(t.numel() * t.element_size() for t in ts if t is not None)
 
     def cache_need(self) -> CacheNeed:
@@ -110,7 +122,7 @@ class LatentAttention(Mixer):
     # ---------------------------------------------------------------- one step
     def forward(self, ctx: StepContext, h: torch.Tensor, cache: CacheView) -> torch.Tensor:
         s, n, H = self.spec, ctx.n_tokens, self.spec.n_heads
-        q_width = H * (s.head_dim + self.rot_dim)
+        q_width = self.q_rank or H * (s.head_dim + self.rot_dim)
         proj = ctx.scratch("latent.in", (n, self.w_in.shape[0]))
         ops.linear(h, self.w_in, proj)
         q = proj[:, :q_width]
@@ -121,12 +133,22 @@ class LatentAttention(Mixer):
             cos, sin = self.position.tables(ctx)
         else:
             cos = sin = ctx.scratch("latent.norope", (n, 0), torch.float32)
+        expand = EXPAND_PROMPTS and not ctx.all_decode and s.window is None and all(start == 0 for start in ctx.host.starts)
+        if self.q_rank:
+            # both latents' norms and the cache rows in one kernel, then the queries' expansion
+            pool = cache.pools["latent"]
+            q_lat = ctx.scratch("latent.q_lat", (n, self.q_rank))
+            kept = self._step_rows(ctx, pool) if expand and s.own_kv else (None, None)
+            ops.latent_norms(q, self.q_norm, q_lat, self.norm_eps, down, self.latent_norm, cos, sin, cache.slots if s.own_kv else None,
+                             pool if s.own_kv else None, self.rank, self.rot_dim, cache.page_size, *kept)
+            q, down = ctx.scratch("latent.q_up", (n, H * (s.head_dim + self.rot_dim))), None
+            ops.linear(q_lat, self.w_q, q)
         # A step that brings only whole prompts (every sequence starts at 0) has all its keys among its own tokens: it
         # expands them once (two products for the step) and attends with keys head_dim + rot_dim wide and values value_dim
         # wide, a third of the absorbed form's arithmetic per (query, key) pair.  Every other step (portions behind a
         # cached part, single tokens) attends over the cached rows in the absorbed form.  A captured step is a step of
         # single tokens and always takes the absorbed form, so nothing here goes stale in a replay.
-        if EXPAND_PROMPTS and not ctx.all_decode and s.window is None and all(start == 0 for start in ctx.host.starts):
+        if expand:
             heads = self._expanded(ctx, q, down, cos, sin, cache)
             if gate is not None:
                 ops.sigmoid_gate(heads.view(n, H * s.value_dim), gate)
@@ -143,8 +165,8 @@ class LatentAttention(Mixer):
         pool = cache.pools["latent"]
         q_full = ctx.scratch("latent.q", (n, H, self.row), torch.float32)
         ops.heads_linear(q.view(n, H, s.head_dim + self.rot_dim)[:, :, :s.head_dim], self.w_uk_t, q_full[:, :, :self.rank])
-        ops.latent_prepare(q, down, self.latent_norm, self.norm_eps, cos, sin, cache.slots if s.own_kv else None,
-                           pool if s.own_kv else None, q_full, H, s.head_dim, self.rot_dim, self.rank, cache.page_size)
+        own = down is not None
+        ops.latent_prepare(q, down, self.latent_norm, self.norm_eps, cos, sin, cache.slots if own else None, pool if own else None, q_full, H, s.head_dim, self.rot_dim, self.rank, cache.page_size)
         mixed = ctx.scratch("latent.mixed", (n, H, self.rank))
         ops.paged_attention_general(ctx, q_full, pool, pool, mixed, cache.block_table, s.scale, s.window, s.chunk, None,
                                     key_width=self.row, value_width=self.rank, sinks=self.sinks)
@@ -152,19 +174,23 @@ class LatentAttention(Mixer):
         ops.heads_linear(mixed, self.w_uv, heads, gate)
         return heads
 
+    def _step_rows(self, ctx, pool):
+        """(latent, rotated key part) of the step's own tokens: the cache's owner fills them, those who borrow its rows read them."""
+        key = ("latent.rows", pool.data_ptr())
+        if key not in ctx.shared:
+            ctx.shared[key] = (ctx.scratch(f"latent.rows.{pool.data_ptr()}", (ctx.n_tokens, self.rank)),
+                               ctx.scratch(f"latent.rot.{pool.data_ptr()}", (ctx.n_tokens, self.rot_dim)))
+        return ctx.shared[key]
+
     def _expanded(self, ctx, q, down, cos, sin, cache) -> torch.Tensor:
         s, n, H = self.spec, ctx.n_tokens, self.spec.n_heads
         pool = cache.pools["latent"]
-        key = ("latent.rows", pool.data_ptr())            # what the cache's owner wrote this step, for those who borrow it
         q_cat = ctx.scratch("latent.q", (n, H, s.head_dim + self.rot_dim), torch.float32)
-        if s.own_kv:
-            latent = ctx.scratch(f"latent.rows.{pool.data_ptr()}", (n, self.rank))
-            shared = ctx.scratch(f"latent.rot.{pool.data_ptr()}", (n, self.rot_dim))
+        latent, shared = self._step_rows(ctx, pool)
+        if down is not None:
             ops.latent_prepare(q, down, self.latent_norm, self.norm_eps, cos, sin, cache.slots, pool, q_cat, H, s.head_dim,
                                self.rot_dim, self.rank, cache.page_size, plain_too=True, latent_out=latent, rot_out=shared)
-            ctx.shared[key] = (latent, shared)
         else:
-            latent, shared = ctx.shared[key]
             ops.latent_prepare(q, None, None, self.norm_eps, cos, sin, None, None, q_cat, H, s.head_dim, self.rot_dim, self.rank,
                                cache.page_size, plain_too=True)
         k_plain = ctx.scratch("latent.k_plain", (n, H * s.head_dim))

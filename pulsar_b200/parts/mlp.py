@@ -137,8 +137,9 @@ class ClampedGLU(FeedForward):
 
 @FEED_FORWARDS.register("mlp")
 class ActivatedMLP(FeedForward):
-    """act(h Wu^T) Wd^T without gate and without bias; ``spec.activation``: "gelu" (the erf form), "gelu_tanh", "silu" or
-    "relu".  The up product leaves float32 rows, the activation runs in float32 and rounds once (``ops.activation``).
+    """act(h Wu^T) Wd^T without gate and without bias; ``spec.activation``: "gelu" (the erf form), "gelu_tanh", "silu", "relu" or
+    "relu2" (max(x, 0)^2).  The up product leaves float32 rows, the activation runs in float32 and rounds once (``ops.activation``);
+    "relu2" runs in the product's epilogue where that fuses (``ops.squared_relu_linear``).
     Options (``spec.extra``): tensor names by role "up", "down"."""
 
     def __init__(self, spec: FeedForwardSpec, prefix: str, dtype: torch.dtype):
@@ -161,10 +162,13 @@ class ActivatedMLP(FeedForward):
 
     def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
         s, n = self.spec, ctx.n_tokens
-        up = ctx.scratch("mlp.up32", (n, s.intermediate), torch.float32)
-        ops.linear(h, self.w_up, up)
         act = ctx.scratch("mlp.act", (n, s.intermediate))
-        ops.activation(up, act, s.activation)
+        if s.activation == "relu2":
+            ops.squared_relu_linear(ctx, h, self.w_up, act)
+        else:
+            up = ctx.scratch("mlp.up32", (n, s.intermediate), torch.float32)
+            ops.linear(h, self.w_up, up)
+            ops.activation(up, act, s.activation)
         out = ctx.scratch("mlp.out", (n, s.hidden))
         ops.linear(act, self.w_down, out)
         return out

@@ -1,4 +1,4 @@
-"""A mixture of gated experts with a sigmoid router and an optional shared expert."""
+"""A mixture of gated or ungated experts with a sigmoid or softmax router and an optional shared expert."""
 from __future__ import annotations
 
 from typing import Dict, List, Optional
@@ -28,8 +28,14 @@ class MixtureOfExperts(FeedForward):
     With ``scoring`` "softmax" the scores are s = softmax(W_r h) over all experts instead of sigmoids, and ``renorm_eps`` is added
     to the chosen scores' sum before a renormalising division.
 
+    With ``gated`` False an expert is W_down max(W_up h, 0)^2 (``spec.activation`` "relu2"; no gate projection).  ``identity`` more
+    outputs of the router stand for experts that return their input and have no tensors.  ``correction`` (a tensor name behind
+    the prefix, one number per router output) joins the scores for the choice, not for the weights.  ``groups`` = (count, keep):
+    the router's outputs form ``count`` groups of neighbours, a group counts as its best choice score, and the chosen come from
+    the ``keep`` best groups.
+
     Options (``spec.extra``): ``experts``, ``top``, ``router_scale``, ``renormalize``, ``scoring``, ``renorm_eps``, ``limit``, ``alpha``, ``shift``,
-    ``weight_input``, ``shared`` (FeedForwardSpec or None), ``shared_prefix`` ("shared."), ``shared_gate``, ``tensor_names``
+    ``gated``, ``identity``, ``correction``, ``groups``, ``weight_input``, ``shared`` (FeedForwardSpec or None), ``shared_prefix`` ("shared."), ``shared_gate``, ``tensor_names``
     by role "router", "gate", "up", "down" (an expert's tensors are ``<prefix>e<i>.<name>``).
 
     The router's choice stays on the device: the kernels take the chosen ids as an array, so a step of single tokens can
@@ -41,8 +47,19 @@ class MixtureOfExperts(FeedForward):
     def __init__(self, spec: FeedForwardSpec, prefix: str, dtype: torch.dtype):
         self.spec, self.prefix, self.dtype = spec, prefix, dtype
         self.n_experts, self.top = int(spec.option("experts", 0)), int(spec.option("top", 0))
-        if not (0 < self.top <= self.n_experts):
-            raise ValueError(f"moe: top ({self.top}) must lie between 1 and the number of experts ({self.n_experts})")
+        self.identity = int(spec.option("identity", 0) or 0)
+        self.outputs = self.n_experts + self.identity          # what the router scores
+        if not (0 < self.top <= self.outputs) or self.n_experts <= 0 or self.identity < 0:
+            raise ValueError(f"moe: top ({self.top}) must lie between 1 and the number of experts ({self.outputs})")
+        self.gated = bool(spec.option("gated", True))
+        if not self.gated and spec.activation != "relu2":
+            raise ValueError(f"moe: ungated experts with activation '{spec.activation}' are not implemented (only 'relu2')")
+        self.groups = spec.option("groups", None)
+        if self.groups is not None:
+            count, keep = (int(v) for v in self.groups)
+            if count <= 0 or self.outputs % count or not (0 < keep <= count) or self.top > keep * (self.outputs // count):
+                raise ValueError(f"moe: {keep} of {count} groups over {self.outputs} router outputs do not offer {self.top} experts")
+            self.groups = (count, keep)
         self.router_scale = float(spec.option("router_scale", 1.0))
         self.renormalize = bool(spec.option("renormalize", False))
         self.scoring = str(spec.option("scoring", "sigmoid"))
@@ -54,6 +71,10 @@ class MixtureOfExperts(FeedForward):
         names = dict(spec.option("tensor_names", ()))
         self.names = {r: names.get(r, d) for r, d in (("router", "router"), ("gate", "gate"), ("up", "up"), ("down", "down"))}
         self.weight_input = bool(spec.option("weight_input", False))
+        if self.weight_input and (self.identity or not self.gated):
+            raise ValueError("moe: weights on the experts' inputs go with gated experts and no identity experts")
+        self.correction_name = prefix + str(spec.option("correction")) if spec.option("correction", None) else None
+        self.correction = None
         shared = spec.option("shared", None)
         self.shared = self.shared_gate_name = None
         if shared is not None:
@@ -69,10 +90,13 @@ class MixtureOfExperts(FeedForward):
         s = self.spec
         specs = []
         for i in range(self.n_experts):
-            specs += [WeightSpec(self._expert(i, "gate"), (s.intermediate, s.hidden)),
-                      WeightSpec(self._expert(i, "up"), (s.intermediate, s.hidden)),
+            if self.gated:
+                specs.append(WeightSpec(self._expert(i, "gate"), (s.intermediate, s.hidden)))
+            specs += [WeightSpec(self._expert(i, "up"), (s.intermediate, s.hidden)),
                       WeightSpec(self._expert(i, "down"), (s.hidden, s.intermediate))]
-        specs.append(WeightSpec(self.prefix + self.names["router"], (self.n_experts, s.hidden), role="vector", init="normal"))
+        specs.append(WeightSpec(self.prefix + self.names["router"], (self.outputs, s.hidden), role="vector", init="normal"))
+        if self.correction_name is not None:
+            specs.append(WeightSpec(self.correction_name, (self.outputs,), role="vector", init="small"))
         if self.shared is not None:
             specs += self.shared.weight_specs()
         if self.shared_gate_name is not None:
@@ -81,8 +105,13 @@ class MixtureOfExperts(FeedForward):
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         n = self.n_experts
-        self.w_gate_up = torch.stack([torch.cat([tensors[self._expert(i, "gate")], tensors[self._expert(i, "up")]], dim=0)
-                                      for i in range(n)]).contiguous()                      # [E, 2 ff, width]
+        if self.gated:
+            self.w_gate_up = torch.stack([torch.cat([tensors[self._expert(i, "gate")], tensors[self._expert(i, "up")]], dim=0)
+                                          for i in range(n)]).contiguous()                  # [E, 2 ff, width]
+        else:
+            self.w_gate_up = torch.stack([tensors[self._expert(i, "up")] for i in range(n)]).contiguous()       # [E, ff, width]
+        if self.correction_name is not None:
+            self.correction = tensors[self.correction_name].contiguous()
         self.w_down = torch.stack([tensors[self._expert(i, "down")] for i in range(n)]).contiguous()    # [E, width, ff]
         self.router = tensors[self.prefix + self.names["router"]].contiguous()
         if self.shared_gate_name is not None:           # one more row of the router's product: it competes for nothing
@@ -102,7 +131,7 @@ class MixtureOfExperts(FeedForward):
         weights = ctx.scratch("moe.weights", (n, top), torch.float32)
         shared_scale = ctx.scratch("moe.shared_scale", (n, 1), torch.float32) if self.shared_gate_name is not None else None
         ops.moe_route(h, self.router, ids, weights, self.router_scale, self.renormalize, shared_scale,
-                      softmax=self.scoring == "softmax", renorm_eps=self.renorm_eps)
+                      softmax=self.scoring == "softmax", renorm_eps=self.renorm_eps, correction=self.correction, groups=self.groups)
         shared = self.shared.forward(ctx, h) if self.shared is not None else None
         act = ctx.scratch("moe.act", (n * top, s.intermediate))
         out = ctx.scratch("moe.out", (n, s.hidden))
@@ -111,8 +140,12 @@ class MixtureOfExperts(FeedForward):
             work = ctx.scratch("moe.work", (ops.moe_grouped_workspace(n, top, self.n_experts),), torch.int32)
             gathered = ctx.scratch("moe.gathered", (n * top, s.hidden)) if ops.MOE_TCGEN05 else None
             ops.moe_grouped(h, self.w_gate_up, self.w_down, ids, weights, shared, act, y, out, work, self.gating, gathered,
-                            weight_input=self.weight_input, add_scale=shared_scale)
+                            weight_input=self.weight_input, add_scale=shared_scale, ungated=not self.gated, identity=self.identity)
             return out
-        ops.moe_gate_up(h, self.w_gate_up, ids, act, self.gating, weights if self.weight_input else None)
-        ops.moe_down(act, self.w_down, ids, None if self.weight_input else weights, shared, out, shared_scale)
+        if self.gated:
+            ops.moe_gate_up(h, self.w_gate_up, ids, act, self.gating, weights if self.weight_input else None)
+        else:
+            ops.moe_up(h, self.w_gate_up, ids, act)
+        ops.moe_down(act, self.w_down, ids, None if self.weight_input else weights, shared, out, shared_scale,
+                     identity=h if self.identity else None)
         return out
