@@ -2,7 +2,8 @@
 
 For each size the design's model and a Qwen3 dense model of the same width, depth, heads, feed-forward size and vocabulary
 (for Megusun and Bumotar: a Topunex model, the closest one, with the same width, depth, projection sizes, experts and vocabulary;
-its entry keeps the key "dense") are built with random weights (bfloat16) and timed through the step function:
+its entry keeps the key "dense"; for Rikolix two models: Topunex with feed-forwards of equal numbers of weights, and under
+"latent" Bumotar for the layers with a latent) are built with random weights (bfloat16) and timed through the step function:
 
   prefill   one step of 2,048 prompt tokens (tokens a second, ms)
   decode    steps of single tokens of 8 requests whose context ends at 2,048 (tokens a second, ms per step)
@@ -170,7 +171,8 @@ def bumotar_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
     n = PROMPT if phase == "prefill" else BATCH
     seqs = 1 if phase == "prefill" else BATCH
     start = 0 if phase == "prefill" else CONTEXT - 1
-    Lp, Ll = BUMOTAR_RUNS.count("parallel"), BUMOTAR_RUNS.count("latent")
+    runs = z.get("runs", BUMOTAR_RUNS)
+    Lp, Ll = runs.count("parallel"), runs.count("latent")
     L, w = Lp + Ll, z["width"]
     H, G, d, rot, rank = z["heads"], z["kv_heads"], z["dim"], z["rot"], z["rank"]
     D, V = z["ret_dim"], z["ret_vdim"]
@@ -210,6 +212,113 @@ def bumotar_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
         "moe_gate_up": (L * (n * top * 2 * fe * w * 2 + n * w * 2), L * 4.0 * n * top * fe * w, "fp32 FMA"),
         "moe_down": (L * (n * top * fe * w * 2 + n * w * 4), L * 2.0 * n * top * fe * w, "fp32 FMA"),
         "silu_mul": (L * n * fs * 6, 0.0, ""),
+    }
+    return {k: (b * steps, f * steps, on) for k, (b, f, on) in work.items()}
+
+
+# Rikolix at sizes that resemble layers of real models: of every four layers one owns a latent of 512 (rotated part 64, queries
+# out of a latent of three eighths of the width) and two borrow it, the third has grouped sigmoid attention (heads of 128, half
+# of each turning, values turning wholly); the feed-forwards alternate between a dense one and 32 experts with four identity
+# outputs in six groups, of which a token uses 4 out of three groups.  What the models beside it need is in the shape too: their
+# gated feed-forwards have three matrices where these have two, so theirs are two thirds as wide.
+RIKOLIX_SIZES = {
+    "1k": dict(width=1024, layers=8, heads=8, kv_heads=2, dim=128, rot=64, rank=512, q_rank=384, window=CONTEXT, keep=0, ret_dim=64,
+               ret_vdim=128, ff=6144, experts=16, identity=2, groups=6, keep_groups=3, top=2, expert_ff=768, shared_ff=0, vocab=32000),
+    "2k": dict(width=2048, layers=8, heads=16, kv_heads=4, dim=128, rot=64, rank=512, q_rank=768, window=CONTEXT, keep=0, ret_dim=64,
+               ret_vdim=128, ff=12288, experts=32, identity=4, groups=6, keep_groups=3, top=4, expert_ff=1536, shared_ff=0, vocab=32000),
+    "4k": dict(width=4096, layers=8, heads=32, kv_heads=8, dim=128, rot=64, rank=512, q_rank=1536, window=CONTEXT, keep=0, ret_dim=64,
+               ret_vdim=128, ff=18432, experts=32, identity=4, groups=6, keep_groups=3, top=4, expert_ff=3072, shared_ff=0, vocab=32000),
+}
+RIKOLIX_LAYERS = [("latent", "dense"), ("borrowed", "moe"), ("attention", "dense"), ("borrowed", "moe")] * 2
+
+
+def rikolix_config(z: dict) -> dict:
+    lat = dict(heads=z["heads"], dim=z["dim"], rot_dim=z["rot"], vdim=z["dim"], q_rank=z["q_rank"], kv_rank=z["rank"],
+               scale=1.0 / math.sqrt(z["dim"] + z["rot"]), rot=dict(base=100000.0, dims=z["rot"]))
+    att = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["dim"], scale=1.0 / math.sqrt(z["dim"]),
+               rot=dict(base=100000.0, dims=z["rot"]))
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"]), router=dict(experts=z["experts"], top=z["top"], identity=z["identity"],
+                                                                       groups=dict(count=z["groups"], keep=z["keep_groups"])))
+    layers, owner = [], 0
+    for i, (kind, ff) in enumerate(RIKOLIX_LAYERS):
+        owner = i if kind == "latent" else owner
+        mixer = dict(att) if kind == "attention" else dict(lat, kv_from=owner) if kind == "borrowed" else dict(lat)
+        layers.append(dict(type="attention" if kind == "attention" else "latent_attention", mixer=mixer,
+                           mlp=dict(kind="dense", ff=z["ff"]) if ff == "dense" else dict(moe)))
+    return dict(architecture="Rikolix", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), embedding=dict(scale=1.0), layers=layers)
+
+
+def rikolix_topunex_config(z: dict) -> dict:
+    """Topunex with as many layers, heads, experts and feed-forward weights (gated units: two thirds as wide), no shared expert."""
+    raw = topunex_config(dict(z, ff=z["ff"] * 2 // 3, expert_ff=z["expert_ff"] * 2 // 3, shared_ff=1))
+    dense, moe = raw["layers"][0]["mlp"], dict(raw["layers"][1]["mlp"])
+    moe.pop("shared")
+    for layer, (_, ff) in zip(raw["layers"], RIKOLIX_LAYERS):
+        layer["mixer"].pop("mask")
+        layer["mlp"] = dict(dense) if ff == "dense" else dict(moe)
+    return raw
+
+
+def rikolix_topunex_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
+    own = topunex_work(dict(z, ff=z["ff"] * 2 // 3, expert_ff=z["expert_ff"] * 2 // 3, layers=8), phase)
+    halves = {"moe_route", "moe_grouped", "moe_gate_up", "moe_down"}          # four routed layers where that table counts seven, four dense where it counts one
+    out = {k: ((b * 4 / 7, f * 4 / 7, on) if k in halves else (b, f, on)) for k, (b, f, on) in own.items() if k != "clamped_glu"}
+    out["glu_bias"] = tuple(4 * v if isinstance(v, float) else v for v in (float(own["glu_bias"][0]), 0.0, ""))
+    return out
+
+
+def rikolix_bumotar_config(z: dict) -> dict:
+    """Bumotar's latent layers in the places of Rikolix's, its parallel layers in those of the attention, experts everywhere."""
+    raw = bumotar_config(dict(z, expert_ff=z["expert_ff"] * 2 // 3, shared_ff=1))
+    par, lat = raw["layers"][0], raw["layers"][1]
+    for layer in (par, lat):
+        layer["mlp"].pop("shared", None)
+    raw["layers"] = [dict(par) if kind == "attention" else dict(lat) for kind, _ in RIKOLIX_LAYERS]
+    raw.pop("loop")
+    return raw
+
+
+def rikolix_bumotar_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
+    return bumotar_work(dict(z, expert_ff=z["expert_ff"] * 2 // 3, runs=["parallel" if kind == "attention" else "latent" for kind, _ in RIKOLIX_LAYERS]), phase)
+
+
+def rikolix_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
+    """Per kernel class of Rikolix: (bytes it must move, flops, what the flops run on) summed over the layers of a step."""
+    n = PROMPT if phase == "prefill" else BATCH
+    seqs = 1 if phase == "prefill" else BATCH
+    start = 0 if phase == "prefill" else CONTEXT - 1
+    kinds = [k for k, _ in RIKOLIX_LAYERS]
+    Lo, La = kinds.count("latent"), kinds.count("attention")
+    Ll, Ld, Lm = Lo + kinds.count("borrowed"), sum(1 for _, f in RIKOLIX_LAYERS if f == "dense"), sum(1 for _, f in RIKOLIX_LAYERS if f == "moe")
+    L, w, H, G, d, rot, rank, qr = len(kinds), z["width"], z["heads"], z["kv_heads"], z["dim"], z["rot"], z["rank"], z["q_rank"]
+    E, top, fe, outputs = z["experts"], z["top"], z["expert_ff"], z["experts"] + z["identity"]
+    steps = 1 if phase == "prefill" else 4
+    row = rank + rot
+    pairs = seqs * _pairs(n // seqs, start)
+    att = (La * (seqs * (start + n // seqs) * G * 2 * d * 2 + n * H * d * (4 + 2)), La * 4.0 * H * d * pairs)
+    if phase == "prefill":
+        lat = (Ll * n * H * ((d + rot) * (4 + 2) + d * 4), Ll * 2.0 * H * (2 * d + rot) * pairs)
+    else:
+        lat = (Ll * (seqs * (start + 1) * row * 2 + n * H * (row * 4 + rank * 2)), Ll * 2.0 * H * (row + rank) * pairs)
+    attention = (att[0] + lat[0], att[1] + lat[1])
+    real = top * E / outputs                              # experts with weights that a token uses, on average
+    distinct = E * (1.0 - (1.0 - top / outputs) ** n)
+    work = {
+        "paged_attention_general_tc": (attention[0], attention[1], "bf16 tensor"),
+        "paged_attention_general_tiled": (attention[0], attention[1], "fp32 FMA"),
+        "paged_attention_general": (attention[0], attention[1], "fp32 FMA"),
+        "qk_prepare_whole": (La * n * ((H + 2 * G) * d * 2 + H * d * 4 + 2 * G * d * 2), 0.0, ""),
+        "latent_norms": (Ll * n * qr * 4 + Lo * n * row * 4, 0.0, ""),
+        "latent_prepare": (Ll * n * H * rot * 6 if phase == "decode" else Ll * n * H * (d + rot) * 6, 0.0, ""),
+        "heads_linear": (Ll * (2 * H * d * rank * 2 + n * H * (d * 2 + rank * 4 + rank * 2 + d * 2)), Ll * 2.0 * n * H * d * rank * 2, "fp32 FMA"),
+        "latent_expand_keys": (Ll * n * H * (2 * d + rot) * 2, 0.0, ""),
+        "post_norm_add": (2 * L * n * w * (2 + 4 + 4 + 2), 0.0, ""),
+        "add_rmsnorm": (n * w * (4 + 2), 0.0, ""),
+        "gemm_tcgen05": (Ld * (z["ff"] * w + n * (w + z["ff"])) * 2, Ld * 2.0 * n * w * z["ff"], "bf16 tensor"),
+        "moe_route": (Lm * (n * w * 2 + outputs * w * 4), 0.0, ""),
+        "moe_grouped": (Lm * (distinct * 2 * w * fe * 2 + n * w * 4 + n * real * (fe * 4 + w * 8)), Lm * 2.0 * n * real * 2 * w * fe, "bf16 tensor"),
+        "moe_up": (Lm * (n * real * fe * w * 2 + n * w * 2), Lm * 2.0 * n * real * fe * w, "fp32 FMA"),
+        "moe_down": (Lm * (n * real * fe * w * 2 + n * w * 4), Lm * 2.0 * n * real * fe * w, "fp32 FMA"),
     }
     return {k: (b * steps, f * steps, on) for k, (b, f, on) in work.items()}
 
@@ -414,30 +523,37 @@ def rooflines(kernels: Dict[str, List[float]], work: Dict[str, Tuple[float, floa
     return out
 
 
-# design -> (sizes, its configuration, its kernels' work, the configuration of the model beside it, that model's kernels' work)
+# design -> (sizes, its configuration, its kernels' work, the configuration of the model beside it, that model's kernels' work[,
+# the same two of a second model beside it])
 DESIGNS = {"bubotar": (SIZES, bubotar_config, own_work, dense_config, like_work),
            "topunex": (TOPUNEX_SIZES, topunex_config, topunex_work, dense_config, like_work),
            "megusun": (MEGUSUN_SIZES, megusun_config, megusun_work, topunex_config, topunex_work),
-           "bumotar": (BUMOTAR_SIZES, bumotar_config, bumotar_work, topunex_config, topunex_work)}
+           "bumotar": (BUMOTAR_SIZES, bumotar_config, bumotar_work, topunex_config, topunex_work),
+           "rikolix": (RIKOLIX_SIZES, rikolix_config, rikolix_work, rikolix_topunex_config, rikolix_topunex_work,
+                       rikolix_bumotar_config, rikolix_bumotar_work)}
 
 
 def run(args, bench) -> dict:
     """``bench``: the bench module (its timing functions, peaks and clock sampler are used as they are)."""
     import torch
     pk = bench.peaks()
-    table, make_config, design_work, beside_config, beside_work = DESIGNS[args.design]
+    table, make_config, design_work, beside_config, beside_work = DESIGNS[args.design][:5]
+    second = DESIGNS[args.design][5:]
     sizes = [s for s in (args.sizes.split(",") if args.sizes else table) if s]
     line = {"design": args.design, "dtype": "bf16", "data": "synthetic: random weights, random token ids, random cache contents for decode",
             "prompt_tokens": PROMPT, "decode": {"batch": BATCH, "context": CONTEXT}, "peaks": pk, "sizes": {}}
     for size in sizes:
         z = table[size]
         entry = {"shape": z}
-        for who, raw in (("design", make_config(z)), ("dense", beside_config(z))):       # "dense": the model beside it (Qwen3 dense, or Topunex for Megusun)
+        # "dense": the model beside it (Qwen3 dense, or Topunex for Megusun, Bumotar and Rikolix)
+        models = [("design", make_config(z), design_work), ("dense", beside_config(z), beside_work)]
+        if second:
+            models.append(("latent", second[0](z), second[1]))
+        for who, raw, work in models:
             engine = build(raw)
             p_seconds = bench.time_prefill(engine, PROMPT)
             d_seconds, _, _ = bench.time_decode(engine, BATCH, CONTEXT, args.steps, max(3, args.warmup))
             prefill_k, decode_k = profiled(engine, bench)
-            work = design_work if who == "design" else beside_work
             entry[who] = {
                 "model": engine.model.spec.architecture, "weights_gb": round(engine.model.weight_bytes(0) / 1e9, 3),
                 "prefill_tokens_per_s": round(PROMPT / p_seconds, 1), "prefill_ms": round(p_seconds * 1e3, 3),

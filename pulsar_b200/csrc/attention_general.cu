@@ -272,6 +272,7 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
                      float* __restrict__ partial, const int* __restrict__ block_table, const int* __restrict__ cu_q,
                      const int* __restrict__ kv_len, const float* __restrict__ slopes, const float* __restrict__ sinks,
                      const TiledShape ts, const PoolBounds bounds) {
+    pdl_wait();         // may have come onto the SMs while the kernel before it was ending: nothing is touched before that one is done
     constexpr int V = Vec<T>::n;
     const GeneralShape& sh = ts.g;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -490,6 +491,7 @@ general_tiled_kernel(const float* __restrict__ q, const T* __restrict__ k_pool, 
 template <typename T>
 __global__ void general_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, const float* __restrict__ sinks,
                                        int n_splits, const GeneralShape sh) {
+    pdl_wait();
     const size_t row = blockIdx.x;
     const int Hq = sh.Hq, Dv = sh.Dv, out_f32 = sh.out_f32;
     const float* pp = partial + row * n_splits * (Dv + 2);
@@ -554,14 +556,13 @@ int launch_tiled(const float* q, const void* k_pool, const void* v_pool, void* o
         allowed = smem;
     }
     dim3 grid(row_tiles, ts.g.Hkv, ts.n_splits);
-    general_tiled_kernel<T, ACC><<<grid, 128, smem, stream>>>(q, (const T*)k_pool, (const T*)v_pool, (T*)out, partial, block_table,
-                                                              cu_q, kv_len, slopes, sinks, ts, pb::pool_bounds_now());
-    int status = launch_status();
+    int status = launch_pdl(general_tiled_kernel<T, ACC>, grid, dim3(128), smem, stream, q, (const T*)k_pool, (const T*)v_pool, (T*)out, partial,
+                            block_table, cu_q, kv_len, slopes, sinks, ts, pb::pool_bounds_now());
     if (status == 0 && ts.n_splits > 1) {
         int b = 32;
         while (b < ts.g.Dv && b < 256) b <<= 1;
-        general_combine_kernel<T><<<n_tokens * ts.g.Hq, b, 0, stream>>>(partial, (T*)out, sinks, ts.n_splits, ts.g);
-        status = launch_status();
+        status = launch_pdl(general_combine_kernel<T>, dim3(n_tokens * ts.g.Hq), dim3(b), 0, stream, (const float*)partial, (T*)out, sinks,
+                            ts.n_splits, ts.g);
     }
     return status;
 }

@@ -107,6 +107,24 @@ __device__ __forceinline__ float gated(float g, float u, const GatedInter& p) {
     return g / (1.0f + expf(-p.alpha * g)) * (u + p.shift);
 }
 
+// Four neighbouring elements at once: 16 bytes of float32, 8 bytes of bfloat16 (the address aligned to as much).
+__device__ __forceinline__ void load_quad(const float* p, float (&v)[4]) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void load_quad(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+    v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+__device__ __forceinline__ void store_quad(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store_quad(__nv_bfloat16* p, const float (&v)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
 // max(x, 0)^2: the activation of ungated feed-forwards that the products' epilogues can apply.
 __device__ __forceinline__ float squared_relu(float x) {
     const float r = fmaxf(x, 0.0f);

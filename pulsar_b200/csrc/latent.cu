@@ -178,7 +178,10 @@ struct NormsShape {
     int q_rank, rank, rot_dim, rot_dims, page_size;
     long q_tok, down_tok;
     float eps;
+    int quads;          // the queries' latent is read and written four elements at a time
 };
+
+constexpr int kNormQuads = 4;       // quads a thread of 128 holds: query latents up to 2,048
 
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -192,6 +195,31 @@ latent_norms_kernel(const T* __restrict__ q_lat, const float* __restrict__ q_nor
     if (blockIdx.y == 0) {
         const T* x = q_lat + (size_t)t * sh.q_tok;
         float ss = 0.0f;
+        if (sh.quads) {                         // uniform over the grid: four elements at a time, the row in registers
+            float v[kNormQuads][4];
+#pragma unroll
+            for (int it = 0; it < kNormQuads; ++it) {
+                const int i = (threadIdx.x + it * blockDim.x) * 4;
+                if (i < sh.q_rank) {
+                    load_quad(x + i, v[it]);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) ss += v[it][e] * v[it][e];
+                }
+            }
+            const float inv = rsqrtf(block_sum(ss, scratch) / (float)sh.q_rank + sh.eps);
+#pragma unroll
+            for (int it = 0; it < kNormQuads; ++it) {
+                const int i = (threadIdx.x + it * blockDim.x) * 4;
+                if (i < sh.q_rank) {
+                    float w[4], y[4];
+                    load_quad(q_norm_w + i, w);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) y[e] = v[it][e] * inv * w[e];
+                    store_quad(q_out + (size_t)t * sh.q_rank + i, y);
+                }
+            }
+            return;
+        }
         for (int i = threadIdx.x; i < sh.q_rank; i += blockDim.x) { const float v = to_float(x[i]); ss += v * v; }
         const float inv = rsqrtf(block_sum(ss, scratch) / (float)sh.q_rank + sh.eps);
         for (int i = threadIdx.x; i < sh.q_rank; i += blockDim.x)
@@ -209,6 +237,7 @@ latent_prepare_kernel(const T* __restrict__ q, const T* __restrict__ down, const
                       const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int* __restrict__ slots,
                       T* __restrict__ pool, float* __restrict__ q_out, T* __restrict__ latent_out, T* __restrict__ rot_out,
                       const PrepareShape sh, const PoolBounds bounds) {
+    pdl_wait();
     __shared__ float scratch[32];
     const int t = blockIdx.x;
     const int rot_dim = sh.rot_dim, half = sh.rot_dims >> 1;
@@ -309,16 +338,13 @@ PB_EXPORT int pb_latent_prepare(int dtype, const void* q, long q_tok, const void
     if (down != nullptr && (norm_w == nullptr || slots == nullptr || pool == nullptr)) return PB_ERR_BAD_SIZE;
     const PrepareShape sh{H, dim, rot_dim, rot_dims, rank, page_size, q_row, q_off, copy_plain, q_tok, down_tok, eps};
     if (dtype == PB_F32)
-        latent_prepare_kernel<float><<<N, 128, 0, stream>>>((const float*)q, (const float*)down, norm_w, cos_t, sin_t, slots,
-                                                            (float*)pool, q_out, (float*)latent_out, (float*)rot_out, sh,
-                                                            pb::pool_bounds_now());
+        return launch_pdl(latent_prepare_kernel<float>, dim3(N), dim3(128), 0, stream, (const float*)q, (const float*)down, norm_w, cos_t, sin_t,
+                          slots, (float*)pool, q_out, (float*)latent_out, (float*)rot_out, sh, pb::pool_bounds_now());
     else if (dtype == PB_BF16)
-        latent_prepare_kernel<__nv_bfloat16><<<N, 128, 0, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)down, norm_w, cos_t,
-                                                                    sin_t, slots, (__nv_bfloat16*)pool, q_out,
-                                                                    (__nv_bfloat16*)latent_out, (__nv_bfloat16*)rot_out, sh,
-                                                                    pb::pool_bounds_now());
-    else return PB_ERR_BAD_DTYPE;
-    return launch_status();
+        return launch_pdl(latent_prepare_kernel<__nv_bfloat16>, dim3(N), dim3(128), 0, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)down,
+                          norm_w, cos_t, sin_t, slots, (__nv_bfloat16*)pool, q_out, (__nv_bfloat16*)latent_out, (__nv_bfloat16*)rot_out, sh,
+                          pb::pool_bounds_now());
+    return PB_ERR_BAD_DTYPE;
 }
 
 // q_lat: rows of q_rank at n * q_tok, normed with q_norm_w (float32 [q_rank]) into q_out [N, q_rank].  down (may be null) and what
@@ -330,7 +356,10 @@ PB_EXPORT int pb_latent_norms(int dtype, const void* q_lat, long q_tok, const fl
     if (N <= 0) return 0;
     if (q_rank <= 0 || rank <= 0 || rot_dim < 0 || rot_dims < 0 || rot_dims > rot_dim || rot_dims % 2 || page_size <= 0) return PB_ERR_BAD_SIZE;
     if (down != nullptr && (norm_w == nullptr || slots == nullptr || pool == nullptr)) return PB_ERR_BAD_SIZE;
-    const NormsShape sh{q_rank, rank, rot_dim, rot_dims, page_size, q_tok, down_tok, eps};
+    const size_t quad = dtype == PB_F32 ? 16 : 8;
+    const bool quads = q_rank % 4 == 0 && q_rank <= kNormQuads * 4 * 128 && q_tok % 4 == 0 && (uintptr_t)q_lat % quad == 0 &&
+                       (uintptr_t)q_out % quad == 0 && (uintptr_t)q_norm_w % 16 == 0;
+    const NormsShape sh{q_rank, rank, rot_dim, rot_dims, page_size, q_tok, down_tok, eps, quads};
     const dim3 grid(N, down != nullptr ? 2 : 1);
     if (dtype == PB_F32)
         return launch_pdl(latent_norms_kernel<float>, grid, dim3(128), 0, stream, (const float*)q_lat, q_norm_w, (float*)q_out,

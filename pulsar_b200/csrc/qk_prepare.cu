@@ -15,8 +15,8 @@
 //   qk_prepare_whole   the same place where q and k are normed over their whole projections: per token the RMS norm runs over
 //                  all Hq*D query elements (and over all Hkv*D key elements) at once with a weight for each, the heads then
 //                  turn (pairs of neighbours or rotate-half), and the value heads may turn too, over `v_rotary` of their Dv
-//                  dimensions with a table of their own.  One block per (token, section q | k | v), the section's row in
-//                  shared memory.
+//                  dimensions with a table of their own.  One block per (token, section q | k | v); the section's row sits in
+//                  registers, four neighbouring elements at a time, where the sizes allow it, else in shared memory.
 //   add_bias       x[n, c] += bias[c] (bias float32): a projection's bias where no kernel behind the product takes it along.
 //   sigmoid_gate_strided   x[n, c] *= sigmoid(gate[n, c / group]) with float32 arithmetic; gate float32 or T, a column slice
 //                  of a wider row; `group` columns of x share a gate column (a gate per head).
@@ -160,6 +160,69 @@ __global__ void qk_prepare_whole_kernel(const TIn* __restrict__ rows, long row_s
     }
 }
 
+// The same for sizes and rows in fours (pairs of neighbours): a thread holds ITERS quads of the section's row in registers.
+template <typename TIn, typename T, int ITERS>
+__global__ void qk_prepare_whole_quads_kernel(const TIn* __restrict__ rows, long row_stride, const float* __restrict__ q_norm_w,
+                                              const float* __restrict__ k_norm_w, const float* __restrict__ cos_t,
+                                              const float* __restrict__ sin_t, const float* __restrict__ v_cos,
+                                              const float* __restrict__ v_sin, float* __restrict__ q_out, T* __restrict__ k_pool,
+                                              T* __restrict__ v_pool, const int* __restrict__ slots, const WholeShape sh,
+                                              const PoolBounds bounds) {
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x, section = blockIdx.y;      // 0: queries, 1: keys, 2: values
+    const int heads = section == 0 ? sh.Hq : section == 1 ? sh.Hkv : sh.Hv, D = section == 2 ? sh.Dv : sh.D;
+    const int n = heads * D;
+    const size_t first = section == 0 ? 0 : (size_t)sh.Hq * sh.D + (section == 2 ? (size_t)sh.Hkv * sh.D : 0);
+    int slot = 0;
+    if (section != 0) {
+        slot = slots[t];
+        if (slot < 0 || !slot_ok(slot, sh.page_size, bounds)) return;        // uniform over the block
+    }
+    const TIn* src = rows + (size_t)t * row_stride + first;
+    float x[ITERS][4];
+    float ss = 0.0f;
+#pragma unroll
+    for (int it = 0; it < ITERS; ++it) {
+        const int i = (threadIdx.x + it * blockDim.x) * 4;
+        if (i < n) {
+            load_quad(src + i, x[it]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) ss += x[it][e] * x[it][e];
+        }
+    }
+    const float* w = section == 0 ? q_norm_w : section == 1 ? k_norm_w : nullptr;
+    float r = 1.0f;
+    if (w != nullptr) r = rsqrtf(block_sum(ss, scratch) / (float)n + sh.eps);
+    const int rotary = section == 2 ? sh.v_rotary : sh.rotary, turning = rotary >> 1;
+    const float* c = (section == 2 ? v_cos : cos_t) + (size_t)t * turning;
+    const float* s = (section == 2 ? v_sin : sin_t) + (size_t)t * turning;
+    const size_t page = (size_t)(slot / sh.page_size), in_page = slot % sh.page_size;
+#pragma unroll
+    for (int it = 0; it < ITERS; ++it) {
+        const int i = (threadIdx.x + it * blockDim.x) * 4;
+        if (i >= n) continue;
+        const int head = i / D, at = i - head * D;
+        float y[4] = {x[it][0], x[it][1], x[it][2], x[it][3]};
+        if (w != nullptr) {
+            float wv[4];
+            load_quad(w + i, wv);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] = y[e] * r * wv[e];
+        }
+        if (at < rotary) {                               // both pairs of the quad turn (rotary is a multiple of 4)
+            const float2 cc = *reinterpret_cast<const float2*>(c + (at >> 1)), sn = *reinterpret_cast<const float2*>(s + (at >> 1));
+            const float u0 = y[0], u1 = y[2];
+            y[0] = u0 * cc.x - y[1] * sn.x;
+            y[1] = y[1] * cc.x + u0 * sn.x;
+            y[2] = u1 * cc.y - y[3] * sn.y;
+            y[3] = y[3] * cc.y + u1 * sn.y;
+        }
+        if (section == 0) store_quad(q_out + (size_t)t * n + i, y);
+        else store_quad((section == 1 ? k_pool : v_pool) + ((page * heads + head) * sh.page_size + in_page) * D + at, y);
+    }
+}
+
 template <typename TIn, typename T>
 int launch_whole(const void* rows, long row_stride, const float* q_norm_w, const float* k_norm_w, const float* cos_t, const float* sin_t,
                  const float* v_cos, const float* v_sin, float* q_out, void* k_pool, void* v_pool, const int* slots, int n,
@@ -167,6 +230,21 @@ int launch_whole(const void* rows, long row_stride, const float* q_norm_w, const
     int widest = sh.Hq * sh.D;
     if (sh.Hkv * sh.D > widest) widest = sh.Hkv * sh.D;
     if (sh.Hv * sh.Dv > widest) widest = sh.Hv * sh.Dv;
+    auto aligned = [](const void* p, size_t bytes) { return ((uintptr_t)p % bytes) == 0; };
+    const bool quads = sh.neighbours && sh.D % 4 == 0 && sh.Dv % 4 == 0 && sh.rotary % 4 == 0 && sh.v_rotary % 4 == 0 && row_stride % 4 == 0 &&
+                       aligned(rows, 4 * sizeof(TIn)) && aligned(q_out, 16) && aligned(k_pool, 4 * sizeof(T)) && aligned(v_pool, 4 * sizeof(T)) &&
+                       aligned(q_norm_w, 16) && aligned(k_norm_w, 16) && aligned(cos_t, 8) && aligned(sin_t, 8) && aligned(v_cos, 8) && aligned(v_sin, 8);
+    if (quads && widest <= 4 * 4 * 1024) {
+        const int n_quads = widest / 4, iters = n_quads > 2048 ? 4 : n_quads > 256 ? 2 : 1;
+        const int threads_q = ((n_quads + iters - 1) / iters + 31) / 32 * 32;
+#define PB_QUADS(ITERS) return launch_pdl(qk_prepare_whole_quads_kernel<TIn, T, ITERS>, dim3(n, sh.Hkv > 0 ? 3 : 1), dim3(threads_q), 0, stream,     \
+                                          (const TIn*)rows, row_stride, q_norm_w, k_norm_w, cos_t, sin_t, v_cos, v_sin, q_out, (T*)k_pool, \
+                                          (T*)v_pool, slots, sh, pool_bounds_now())
+        if (iters == 1) PB_QUADS(1);
+        if (iters == 2) PB_QUADS(2);
+        PB_QUADS(4);
+#undef PB_QUADS
+    }
     const size_t smem = sizeof(float) * (size_t)widest;
     if (smem > 200 * 1024) return PB_ERR_TOO_LARGE;
     static size_t allowed = 48 * 1024;                     // per instantiation

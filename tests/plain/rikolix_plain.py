@@ -116,6 +116,23 @@ def choose(scores: torch.Tensor, correction: torch.Tensor, top: int, groups: Opt
     return out
 
 
+def choice_margin(row: List[float], chosen: List[int], groups: Optional[dict]) -> float:
+    """How far the choice score of the last output chosen lies above the best one passed over, and that of the worst group
+    kept above the best group left out (the smaller of the two): what a rounding of the scores must stay below."""
+    E = len(row)
+    allowed, margin = list(range(E)), float("inf")
+    if groups is not None:
+        size = E // int(groups["count"])
+        best = sorted((max(row[g * size:(g + 1) * size]), g) for g in range(int(groups["count"])))[::-1]
+        keep = int(groups["keep"])
+        if keep < len(best):
+            margin = best[keep - 1][0] - best[keep][0]
+        kept = [g for _, g in best[:keep]]
+        allowed = [e for e in allowed if e // size in kept]
+    rest = [row[e] for e in allowed if e not in chosen]
+    return min(margin, min(row[e] for e in chosen) - max(rest)) if rest else margin
+
+
 def mixture(h: torch.Tensor, w: Dict[str, torch.Tensor], mlp: dict, log: Optional[list] = None) -> torch.Tensor:
     """Weighted sum of the chosen experts; outputs of the router behind the experts stand for the input itself."""
     router = mlp["router"]
@@ -123,7 +140,8 @@ def mixture(h: torch.Tensor, w: Dict[str, torch.Tensor], mlp: dict, log: Optiona
     scores = torch.softmax(h @ w["router"].T, dim=-1)
     ids = choose(scores, w["correction"], int(router["top"]), router.get("groups"))
     if log is not None:
-        log.append((scores, ids))
+        choice = (scores + w["correction"]).tolist()
+        log.append(torch.tensor([choice_margin(choice[t], ids[t], router.get("groups")) / max(scores[t].tolist()) for t in range(len(ids))]))
     out = torch.zeros_like(h)
     for t, chosen in enumerate(ids):
         for e in chosen:
@@ -139,7 +157,8 @@ def _under(weights: Dict[str, torch.Tensor], prefix: str) -> Dict[str, torch.Ten
 
 def forward(raw: dict, weights: Dict[str, torch.Tensor], tokens: List[int], dtype=torch.float64, streams: Optional[list] = None,
             log: Optional[list] = None) -> torch.Tensor:
-    """Logits [L, vocab].  ``streams`` receives the residual stream behind every layer, ``log`` (scores, chosen) of every router."""
+    """Logits [L, vocab].  ``streams`` receives the residual stream behind every layer, ``log`` every router's margins
+    (``choice_margin`` over the largest score, per token)."""
     W = {k: v.to(dtype) for k, v in weights.items()}
     eps = float(raw["norm"]["eps"])
     x = W["embed"][torch.tensor(tokens)] * float(raw["embedding"]["scale"])
