@@ -62,6 +62,7 @@ class MixerSpec:
     fixed_sink: Optional[float] = None   # the same with one given number for all heads instead of a learned tensor (0: one is added)
     bias: bool = False               # the q, k, v and o projections have biases (the weight's name + ".b" unless named by role)
     output_gate: bool = False        # the concatenated heads are multiplied by sigmoid(W_g h) before the output projection
+    gate_per_head: bool = False      # a head is multiplied by sigmoid(<its row of W_g, h>), one number per head and token, before the output projection
     values_from_keys: bool = False   # no v projection: the value is the key as projected (before rotation and norm)
     qk_norm_weight: bool = True      # False: q and k are divided by their root mean square (qk_norm_eps) without a weight
     qk_norm_after_rotation: bool = False   # the per-head norm of q and k follows the rotation instead of preceding it

@@ -5,6 +5,7 @@
 //                  chosen s * scale.  ids int32 [N, top] in descending order of s, weights float32 [N, top].
 //                  With `softmax` the scores are s = softmax(z) over all experts instead, and a renormalised weight is
 //                  s / (sum of the chosen s + renorm_eps) * scale.
+//                  With `logit_bias` (float32 [E]) the experts' logits are z + logit_bias[e] throughout.
 //                  With `correction` (float32 [E]) the choice goes by s + correction[e], the weights by s alone.  With
 //                  keep_groups < n_groups the experts form n_groups groups of neighbours of equal size, a group counts as its
 //                  best choice score, and only experts of the keep_groups best groups can be chosen.
@@ -38,10 +39,11 @@ __device__ __forceinline__ void load_chunk(const __nv_bfloat16* p, float (&f)[8]
     for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(u[i] << 16); f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u); }
 }
 // What the choice goes by besides the scores: a number added to each (or null), and how many of the groups of neighbours
-// the chosen experts may come from (keep >= n_groups: all).
+// the chosen experts may come from (keep >= n_groups: all).  logit_bias (or null) joins the logits before they are scored.
 struct RouteChoice {
     const float* correction;
     int n_groups, keep;
+    const float* logit_bias;
 };
 
 constexpr int kRouteRows = 4;            // router rows a warp walks side by side: their loads are in flight together
@@ -148,7 +150,8 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
         for (int r = 0; r < kRouteRows; ++r) {
 #pragma unroll
             for (int k = 0; k < TOK; ++k) {
-                const float zk = warp_sum(z[r][k]);
+                float zk = warp_sum(z[r][k]);
+                if (choice.logit_bias != nullptr && e0 + r < n_experts) zk += choice.logit_bias[e0 + r];
                 if (lane == 0 && e0 + r < n_rows)
                     s[k * n_rows + e0 + r] = (softmax && e0 + r < n_experts) ? zk : 1.0f / (1.0f + expf(-zk));
             }
@@ -358,17 +361,17 @@ int dispatch_route(const void* h, const float* router, int* ids, float* weights,
 
 }  // namespace
 
-// correction (float32 [n_experts] or null) joins the scores for the choice; n_groups groups of neighbours, keep_groups of them
+// logit_bias (float32 [n_experts] or null) joins the experts' logits.  correction (float32 [n_experts] or null) joins the scores for the choice; n_groups groups of neighbours, keep_groups of them
 // open to the choice (1, 1: all experts).
 // router [n_experts + n_extra, width]: the rows behind the experts' are scored too (sigmoid) and go to extra [n, n_extra].
 PB_EXPORT int pb_moe_route(int dtype, const void* h, const float* router, int* ids, float* weights, int n, int width, int n_experts,
                            int top, float scale, int renormalize, int n_extra, float* extra, int softmax, float renorm_eps,
-                           const float* correction, int n_groups, int keep_groups, cudaStream_t stream) {
+                           const float* correction, int n_groups, int keep_groups, const float* logit_bias, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (n_groups <= 0 || keep_groups <= 0 || n_experts % n_groups ||
         (keep_groups < n_groups && (long)keep_groups * (n_experts / n_groups) < top))
         return PB_ERR_BAD_SIZE;
-    const RouteChoice choice{correction, n_groups, keep_groups};
+    const RouteChoice choice{correction, n_groups, keep_groups, logit_bias};
     if (width <= 0 || n_experts <= 0 || top <= 0 || top > n_experts || n_extra < 0 || (n_extra > 0 && extra == nullptr)) return PB_ERR_BAD_SIZE;
     if (dtype == PB_F32) return dispatch_route<float>(h, router, ids, weights, n, width, n_experts, top, scale, renormalize, n_extra, extra, softmax, renorm_eps, choice, stream);
     if (dtype == PB_BF16)

@@ -31,9 +31,9 @@ using namespace pb;
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 
-template <typename T>
+template <typename TIn, typename T>
 __global__ void __launch_bounds__(256)
-causal_conv_silu_kernel(const T* __restrict__ in, long in_tok, const float* __restrict__ taps, const float* __restrict__ bias,
+causal_conv_silu_kernel(const TIn* __restrict__ in, long in_tok, const float* __restrict__ taps, const float* __restrict__ bias,
                         const float* __restrict__ arena, long slot_stride, long tail_offset, const int* __restrict__ cu_q,
                         const int* __restrict__ seq_of_token, const int* __restrict__ state_slots, T* __restrict__ out,
                         int channels, int n_taps) {
@@ -470,24 +470,22 @@ int dispatch_scan(const void* x, const void* xz, const void* proj, const void* w
 
 }  // namespace
 
-// in: rows of the input projection, channel c of token t at in + t * in_tok + c.  out [N, channels].
+// in: rows of the input projection (in_dtype: `dtype` or float32), channel c of token t at in + t * in_tok + c.  out [N, channels].
 // arena: float32, slot s at arena + s * slot_stride, its convolution tail [channels, taps - 1] at tail_offset.
-PB_EXPORT int pb_causal_conv_silu(int dtype, const void* in, long in_tok, const float* taps, const float* bias, const float* arena,
+PB_EXPORT int pb_causal_conv_silu(int in_dtype, int dtype, const void* in, long in_tok, const float* taps, const float* bias, const float* arena,
                                   long slot_stride, long tail_offset, const int* cu_q, const int* seq_of_token,
                                   const int* state_slots, void* out, int n_tokens, int channels, int n_taps, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (channels <= 0 || n_taps < 1) return PB_ERR_BAD_SIZE;
     dim3 grid(n_tokens, (channels + 255) / 256);
     if (grid.y > 65535) return PB_ERR_TOO_LARGE;
-    if (dtype == PB_F32)
-        launch_pdl(causal_conv_silu_kernel<float>, grid, 256, 0, stream, (const float*)in, in_tok, taps, bias, arena, slot_stride, tail_offset,
-                                                                 cu_q, seq_of_token, state_slots, (float*)out, channels, n_taps);
-    else if (dtype == PB_BF16)
-        launch_pdl(causal_conv_silu_kernel<__nv_bfloat16>, grid, 256, 0, stream, (const __nv_bfloat16*)in, in_tok, taps, bias, arena,
-                                                                         slot_stride, tail_offset, cu_q, seq_of_token, state_slots,
-                                                                         (__nv_bfloat16*)out, channels, n_taps);
-    else return PB_ERR_BAD_DTYPE;
-    return launch_status();
+#define PB_CONV(TI, T) return launch_pdl(causal_conv_silu_kernel<TI, T>, grid, dim3(256), 0, stream, (const TI*)in, in_tok, taps, bias, arena, \
+                                         slot_stride, tail_offset, cu_q, seq_of_token, state_slots, (T*)out, channels, n_taps)
+    if (in_dtype == PB_F32 && dtype == PB_F32) PB_CONV(float, float);
+    if (in_dtype == PB_BF16 && dtype == PB_BF16) PB_CONV(__nv_bfloat16, __nv_bfloat16);
+    if (in_dtype == PB_F32 && dtype == PB_BF16) PB_CONV(float, __nv_bfloat16);
+#undef PB_CONV
+    return PB_ERR_BAD_DTYPE;
 }
 
 // x [N, inner] (the convolution's output), xz [N, xz_tok] (the input projection: convolution inputs in columns

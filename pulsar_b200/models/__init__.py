@@ -1,5 +1,5 @@
 """Model assembly.  Importing this package registers the built-in architectures."""
-from . import bubotar, bumotar, megusun, qwen3, rikolix, topunex  # noqa: F401
+from . import bosenex, bubotar, bumotar, megusun, qwen3, rikolix, topunex  # noqa: F401
 from .decoder import DecoderModel
 
 

@@ -96,7 +96,7 @@ _SIGNATURES = {
     "pb_latent_norms": [_I, _P, _L, _P, _P, _P, _L, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "pb_latent_expand_keys": [_I, _P, _P, _P, _I, _I, _I, _I, _P],
     "pb_sigmoid_gate": [_I, _P, _P, _L, _I, _I, _P],
-    "pb_causal_conv_silu": [_I, _P, _L, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _P],
+    "pb_causal_conv_silu": [_I, _I, _P, _L, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _I, _I, _P],
     "pb_selective_scan": [_I, _P, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "pb_selective_scan_prompt_supported": [_I],
     "pb_selective_scan_chunked_supported": [_I],
@@ -110,7 +110,7 @@ _SIGNATURES = {
     "pb_qk_prepare_whole": [_I, _I, _P, _L, _P, _P, _F, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 10 + [_P],
     "pb_sigmoid_gate_strided": [_I, _I, _P, _P, _L, _I, _I, _I, _P],
     "pb_add_bias": [_I, _P, _P, _I, _I, _P],
-    "pb_moe_route": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _I, _F, _P, _I, _I, _P],
+    "pb_moe_route": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _I, _F, _P, _I, _I, _P, _P],
     "pb_moe_gate_up": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     "pb_moe_up": [_I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "pb_moe_down": [_I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _I, _P],
@@ -128,7 +128,14 @@ _SIGNATURES = {
     "pb_retention": [_I, _P, _L, _P, _P, _P, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P],
     "pb_scaled_sum": [_I, _I, _P, _P, _P, _F, _F, ctypes.c_longlong, _P],
     "pb_concat_streams": [_I, _P, _P, _P, _P, _I, _I, _P],
+    "pb_normed_sum": [_I, _P, _P, _P, _P, _P, _F, _F, _I, _I, _F, _P],
+    "pb_recurrence_chunk": [],
+    "pb_recurrence_supported": [_I, _I],
+    "pb_recurrence_workspace": [_I, _I, _I, _I, _I, _I],
+    "pb_matrix_memory": [_I, _P, _L, _P, _P, _F, _P, _F, _F, _F, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "pb_state_space": [_I, _P, _L, _P, _P, _I, _P, _P, _P, _P, _I, _F, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
 }
+_RETURNS = {"pb_recurrence_workspace": _L}        # the others return an int
 _fns = {}
 # the entry points that launch kernels (the others answer questions on the host): what PULSAR_PROF=1 times
 _LAUNCHERS = {"embed", "scale_cap", "move_ids", "add_rmsnorm", "rope_table", "qk_norm_rope_write", "silu_mul", "gather_words",
@@ -139,7 +146,7 @@ _LAUNCHERS = {"embed", "scale_cap", "move_ids", "add_rmsnorm", "rope_table", "qk
               "paged_attention_general", "paged_attention_general_tiled", "paged_attention_general_tc", "qkv_split_write", "heads_linear", "latent_prepare", "latent_norms", "latent_expand_keys", "sigmoid_gate", "causal_conv_silu",
               "selective_scan", "selective_scan_prompt", "selective_scan_chunked", "post_norm_add", "clamped_glu",
               "post_norm_add_bias", "glu_bias", "qk_prepare", "qk_prepare_whole", "sigmoid_gate_strided", "add_bias", "moe_route", "moe_gate_up", "moe_up", "moe_down", "moe_grouped",
-              "norm_shift", "parallel_add", "activation", "min_gru", "diff_combine", "retention", "scaled_sum", "concat_streams"}
+              "norm_shift", "parallel_add", "activation", "min_gru", "diff_combine", "retention", "scaled_sum", "concat_streams", "normed_sum", "matrix_memory", "state_space"}
 
 
 class KernelError(RuntimeError):
@@ -151,7 +158,7 @@ def fn(name: str):
     if f is None:
         f = getattr(library(), name)
         f.argtypes = _SIGNATURES[name]
-        f.restype = ctypes.c_int
+        f.restype = _RETURNS.get(name, ctypes.c_int)
         if profiling.ENABLED and name[3:] in _LAUNCHERS:
             f = profiling.timed_launcher(name, f)
         _fns[name] = f
@@ -688,7 +695,8 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
 
 def gated_linear(ctx, a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, gating=None) -> None:
     """out [M, I] = silu(a Wg^T) * (a Wu^T) with ``w_gate_up`` = gate rows then up rows; with ``gating`` = (limit, alpha,
-    shift) the clamped form g * sigmoid(alpha * g) * (u + shift), g = min(a Wg^T, limit), u = clamp(a Wu^T, -limit, limit).
+    shift) the clamped form g * sigmoid(alpha * g) * (u + shift), g = min(a Wg^T, limit), u = clamp(a Wu^T, -limit, limit)
+    (alpha infinite: max(g, 0) * (u + shift)).
     In bfloat16, up to 16 rows (the weight-streaming kernel) and more than 128 rows (the tcgen05 kernel)
     take one kernel that never writes the [M, 2I] intermediate; otherwise the product followed by the
     gating kernel."""
@@ -705,10 +713,10 @@ def gated_linear(ctx, a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tenso
     linear(a, w_gate_up, gate_up)
     if gating is None:
         silu_mul(gate_up, out)
-    else:
-        if gating[2] != 1.0:
-            raise KernelError("gated_linear: the gating kernel of the unfused path adds 1 to the clamped up part")
+    elif gating[2] == 1.0:
         clamped_glu(gate_up, out, gating[0], gating[1])
+    else:
+        glu_bias(gate_up, None, out, gating)
 
 
 _FORCED_SPLITS = int(os.environ.get("PULSAR_DECODE_SPLITS", "0") or 0)      # > 0: this many splits, for measurements
@@ -1192,14 +1200,16 @@ def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> None:
 # ---------------------------------------------------------------- selective scan
 def causal_conv_silu(ctx, xz: torch.Tensor, channels: int, taps: torch.Tensor, bias: torch.Tensor, arena: torch.Tensor,
                      tail_offset: int, out: torch.Tensor) -> None:
-    """out [N, channels] = silu(causal convolution per channel) of the first ``channels`` columns of ``xz``; inputs before a
-    portion's start come from the sequence's slot of ``arena`` (float32 [slots, floats]; the tail [channels, taps - 1] at
-    ``tail_offset``).  ``taps`` float32 [channels, T], the last column weighs the current token."""
-    _cuda(xz, taps, bias, arena, out)
+    """out [N, channels] = silu(causal convolution per channel) of the first ``channels`` columns of ``xz`` (of ``out``'s dtype or
+    float32; a column slice of a wider tensor will do); inputs before a portion's start come from the sequence's slot of
+    ``arena`` (float32 [slots, floats]; the tail [channels, taps - 1] at ``tail_offset``).  ``taps`` float32 [channels, T], the
+    last column weighs the current token."""
+    _cuda(taps, bias, arena, out)
     n = xz.shape[0]
     assert taps.dtype == bias.dtype == arena.dtype == torch.float32 and taps.shape[0] == channels and bias.numel() == channels
-    assert out.shape == (n, channels) and out.dtype == xz.dtype and xz.shape[1] >= channels and arena.dim() == 2
-    check(fn("pb_causal_conv_silu")(code(xz.dtype), _p(xz), xz.shape[1], _p(taps), _p(bias), _p(arena), arena.shape[1],
+    assert out.shape == (n, channels) and xz.dtype in (out.dtype, torch.float32) and xz.shape[1] >= channels and arena.dim() == 2
+    assert xz.is_cuda and xz.stride(1) == 1
+    check(fn("pb_causal_conv_silu")(code(xz.dtype), code(out.dtype), _p(xz), xz.stride(0), _p(taps), _p(bias), _p(arena), arena.shape[1],
                                     int(tail_offset), _p(ctx.cu_q), _p(ctx.seq_of_token), _p(ctx.state_slots), _p(out), n, channels,
                                     taps.shape[1], stream()), "causal_conv_silu")
 
@@ -1402,15 +1412,16 @@ def add_bias(x: torch.Tensor, bias: torch.Tensor) -> None:
 # ---------------------------------------------------------------- mixture of experts
 def moe_route(h: torch.Tensor, router: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, scale: float = 1.0,
               renormalize: bool = False, extra: Optional[torch.Tensor] = None, softmax: bool = False, renorm_eps: float = 0.0,
-              correction: Optional[torch.Tensor] = None, groups: Optional[Tuple[int, int]] = None) -> None:
+              correction: Optional[torch.Tensor] = None, groups: Optional[Tuple[int, int]] = None,
+              logit_bias: Optional[torch.Tensor] = None) -> None:
     """ids [N, top] int32 and weights [N, top] float32 of the ``top`` largest sigmoid(router @ h) per token (float32 sums;
     ties go to the lower index), weights times ``scale`` (after division by their sum with ``renormalize``).  With ``extra``
     (float32 [N, X]) the router has X more rows behind the experts' that compete for nothing: their sigmoids go there.
     ``softmax``: the scores are softmax(router @ h) over all experts instead; ``renorm_eps`` is added to the chosen scores' sum
     before the division.  ``correction`` (float32 [E]): the choice goes by score + correction, the weights by the score alone.
     ``groups`` = (count, keep): the experts form ``count`` groups of neighbours, a group counts as its best choice score, and
-    only experts of the ``keep`` best groups can be chosen."""
-    _cuda(h, router, ids, weights, extra, correction)
+    only experts of the ``keep`` best groups can be chosen.  ``logit_bias`` (float32 [E]) joins the experts' logits."""
+    _cuda(h, router, ids, weights, extra, correction, logit_bias)
     n, width = h.shape
     n_extra = 0 if extra is None else extra.shape[1]
     e = router.shape[0] - n_extra
@@ -1419,10 +1430,11 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, ids: torch.Tensor, weights:
     assert weights.dtype == torch.float32 and weights.shape == (n, top)
     assert extra is None or (extra.dtype == torch.float32 and extra.shape == (n, n_extra))
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == e)
+    assert logit_bias is None or (logit_bias.dtype == torch.float32 and logit_bias.numel() == e)
     n_groups, keep = (1, 1) if groups is None else (int(groups[0]), int(groups[1]))
     check(fn("pb_moe_route")(code(h.dtype), _p(h), _p(router), _p(ids), _p(weights), n, width, e, top, float(scale),
                              1 if renormalize else 0, n_extra, _p(extra), 1 if softmax else 0, float(renorm_eps), _p(correction), n_groups,
-                             keep, stream()), "moe_route")
+                             keep, _p(logit_bias), stream()), "moe_route")
 
 
 def moe_gate_up(h: torch.Tensor, w_gate_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor, gating,
@@ -1659,6 +1671,97 @@ def scaled_sum(x: torch.Tensor, y: torch.Tensor, out: torch.Tensor, a: float, b:
     assert x.shape == y.shape == out.shape and x.dtype == y.dtype
     check(fn("pb_scaled_sum")(code(x.dtype), code(out.dtype), _p(x), _p(y), _p(out), float(a), float(b), x.numel(), stream()),
           "scaled_sum")
+
+
+def normed_sum(x: torch.Tensor, y: torch.Tensor, wx: torch.Tensor, wy: torch.Tensor, eps: float, out: torch.Tensor, a: float, b: float) -> None:
+    """out = a * rmsnorm(x) * wx + b * rmsnorm(y) * wy row by row (float32 arithmetic, one rounding); ``x`` and ``y`` float32
+    [N, width], ``wx`` and ``wy`` float32 [width]."""
+    _cuda(x, y, wx, wy, out)
+    n, width = out.shape
+    assert x.shape == y.shape == out.shape and x.dtype == y.dtype == wx.dtype == wy.dtype == torch.float32 and wx.numel() == wy.numel() == width
+    check(fn("pb_normed_sum")(code(out.dtype), _p(x), _p(y), _p(wx), _p(wy), _p(out), float(a), float(b), n, width, float(eps), stream()),
+          "normed_sum")
+
+
+# ---------------------------------------------------------------- recurrences whose state decays by one factor per token and head
+RECURRENCE_CHUNKED_MIN = 32    # bfloat16: portions of at least this many tokens take the form in chunks, on the tensor cores
+
+
+def _recurrence_form(ctx, dtype: torch.dtype, key_dim: int, value_dim: int, chunked: Optional[bool]) -> Tuple[bool, int]:
+    """(the form in chunks?, bits of what the kernels take).  A function of the step's shape, the sizes and the dtype alone."""
+    can = fn("pb_recurrence_supported")(key_dim, value_dim)
+    in_chunks = bool(can & 2) and dtype == torch.bfloat16
+    if chunked is None:
+        chunked = in_chunks and (ctx.max_q_len >= RECURRENCE_CHUNKED_MIN or not can & 1)
+    if not (in_chunks if chunked else can & 1):
+        raise KernelError(f"recurrence: keys of {key_dim} and values of {value_dim} in {dtype} do not fit the kernels")
+    return chunked, can
+
+
+def _recurrence_work(ctx, n: int, n_heads: int, key_dim: int, value_dim: int, chunked: bool, normaliser: bool):
+    max_chunks = 0
+    if chunked:
+        size = fn("pb_recurrence_chunk")()
+        max_chunks = sum(-(-int(q) // size) for q in ctx.host.q_lens)
+    floats = fn("pb_recurrence_workspace")(n, n_heads, key_dim, value_dim, max_chunks, 1 if normaliser else 0)
+    return max_chunks, ctx.scratch("recurrence.work", (floats,), torch.float32)
+
+
+def matrix_memory(ctx, rows: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, gate_cap: float, norm_weight: torch.Tensor, eps: float,
+                  state: torch.Tensor, y: torch.Tensor, n_heads: int, key_dim: int, value_dim: int, q_scale: float, denom_eps: float,
+                  chunked: Optional[bool] = None, whole: Optional[bool] = None) -> None:
+    """The matrix memory with exponential gates over the step's tokens.  ``rows`` float32 [N, >= 2 H (D + V) + 2 H] holds per
+    token q (H*D) | k (H*D) | v (H*V) | g (H*V) | i (H) | f (H).  Per head, with log gates i = cap tanh((i + i_bias) / cap) and f =
+    logsigmoid(cap tanh((f + f_bias) / cap)) and the running maximum m = max(f + m, i): S <- exp(f + m' - m) S + exp(i - m) k v^T, n
+    likewise with k alone (``state`` [slots, >= H*D*V + H*D + H] float32: S | n | m of a sequence), o = S^T q / (max(|n . q|,
+    exp(-m)) + denom_eps) with q times ``q_scale``, and ``y`` [N, H*V] = o / rms(o) * ``norm_weight`` * sigmoid(g).  ``chunked``: None
+    picks the form in chunks for bfloat16 steps with portions of ``RECURRENCE_CHUNKED_MIN`` tokens or more, False never, True
+    always.  ``whole`` False: the token-by-token form in tiles of columns also where one block could hold a head."""
+    _cuda(i_bias, f_bias, norm_weight, y)
+    n = rows.shape[0]
+    H, D, V = int(n_heads), int(key_dim), int(value_dim)
+    assert rows.is_cuda and rows.dtype == torch.float32 and rows.stride(1) == 1 and rows.shape[1] >= 2 * H * (D + V) + 2 * H
+    assert i_bias.dtype == f_bias.dtype == norm_weight.dtype == torch.float32 and i_bias.numel() == f_bias.numel() == H
+    assert norm_weight.numel() == H * V and y.shape == (n, H * V)
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.shape[1] >= H * (D * V + D + 1) and state.stride(1) == 1 and state.is_cuda
+    chunked, can = _recurrence_form(ctx, y.dtype, D, V, chunked)
+    whole = not chunked and bool(can & 4) and whole is not False
+    max_chunks, work = (0, None) if whole else _recurrence_work(ctx, n, H, D, V, chunked, True)
+    check(fn("pb_matrix_memory")(code(y.dtype), _p(rows), rows.stride(0), _p(i_bias), _p(f_bias), float(gate_cap), _p(norm_weight), float(eps),
+                                 float(q_scale), float(denom_eps), _p(state), state.stride(0), _p(ctx.cu_q), _p(ctx.state_slots), _p(y), n,
+                                 ctx.n_seqs, H, D, V, 1 if whole else 0, max_chunks, _p(work), stream()), "matrix_memory",
+          kernels=1 if whole else 5 if chunked else 3)
+
+
+def state_space(ctx, rows: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                d_skip: torch.Tensor, norm_weight: torch.Tensor, norm_parts: int, eps: float, state: torch.Tensor, y: torch.Tensor,
+                n_heads: int, n_state: int, value_dim: int, n_groups: int, chunked: Optional[bool] = None) -> None:
+    """The state space with one decay per head over the step's tokens.  ``rows`` float32 [N, >= 2 H*V + 2 G*N + H] holds per token
+    z (H*V) | x (H*V) | B (G*N) | C (G*N) | dt (H).  x, B and C pass the causal convolution (``taps`` [H*V + 2 G*N, T], last column: the
+    current token; ``conv_bias``) and silu; dt = softplus(dt + dt_bias); head h reads B and C of group h // (H / G); S <- exp(-exp(a_log)
+    dt) S + dt B x^T, r = S^T C + d_skip x; ``y`` [N, H*V] = r * silu(z) normed in ``norm_parts`` equal parts * ``norm_weight``.
+    ``state`` [slots, >= H*N*V + (H*V + 2 G*N) (T - 1)] float32: S and the convolution's last inputs of a sequence.  ``chunked`` as for
+    ``matrix_memory``."""
+    _cuda(taps, conv_bias, dt_bias, a_log, d_skip, norm_weight, y)
+    n = rows.shape[0]
+    H, N, V, G = int(n_heads), int(n_state), int(value_dim), int(n_groups)
+    inner, channels, n_taps = H * V, H * V + 2 * G * N, taps.shape[1]
+    assert rows.is_cuda and rows.dtype == torch.float32 and rows.stride(1) == 1 and rows.shape[1] >= inner + channels + H
+    assert taps.dtype == conv_bias.dtype == dt_bias.dtype == a_log.dtype == d_skip.dtype == norm_weight.dtype == torch.float32
+    assert taps.shape[0] == conv_bias.numel() == channels and dt_bias.numel() == a_log.numel() == d_skip.numel() == H
+    assert norm_weight.numel() == inner and inner % int(norm_parts) == 0 and H % G == 0 and y.shape == (n, inner)
+    need = H * N * V + channels * (n_taps - 1)
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.shape[1] >= need and state.is_cuda and state.is_contiguous()
+    chunked, _ = _recurrence_form(ctx, y.dtype, N, V, chunked)
+    xbc = None
+    if chunked:
+        xbc = ctx.scratch("space.xbc", (n, channels), y.dtype)
+        causal_conv_silu(ctx, rows[:, inner:], channels, taps, conv_bias, state, H * N * V, xbc)
+    max_chunks, work = _recurrence_work(ctx, n, H, N, V, chunked, False)
+    check(fn("pb_state_space")(code(y.dtype), _p(rows), rows.stride(0), _p(taps), _p(conv_bias), n_taps, _p(dt_bias), _p(a_log), _p(d_skip),
+                               _p(norm_weight), int(norm_parts), float(eps), _p(state), state.stride(0), _p(ctx.cu_q), _p(ctx.state_slots),
+                               _p(xbc), _p(y), n, ctx.n_seqs, H, N, V, G, max_chunks, _p(work), stream()), "state_space",
+          kernels=5 if chunked else 2)
 
 
 def concat_streams(residual: torch.Tensor, delta: Optional[torch.Tensor], origin: torch.Tensor, out: torch.Tensor) -> None:

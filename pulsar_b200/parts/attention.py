@@ -38,7 +38,8 @@ class Attention(Mixer):
     and ``ops.qk_prepare`` does what stands between it and the attention kernels.  In that form the per-head norm may
     also be the weighted one in front of the rotation (``qk_norm_weight``, not ``qk_norm_after_rotation``), the mixer may
     have a v projection of its own (value heads of ``value_dim``), and the sink may be one given number for all heads
-    (``fixed_sink``; 0 adds one to the softmax's denominator).
+    (``fixed_sink``; 0 adds one to the softmax's denominator).  With ``gate_per_head`` W_g has one row per head, and a head's
+    output is multiplied by the sigmoid of its number.
 
     The differential form (``spec.differential`` = d, part of the general form without rotation, biases or per-head norm):
     every head has two score maps over the same values.  Its query rows hold [map 1 | map 2] (``head_dim`` each) and so do
@@ -67,7 +68,7 @@ class Attention(Mixer):
         # what only ops.qk_prepare does between the projection and the attention kernels (its rows may be wider than
         # q | k, so the gate's columns ride along in the same product)
         self.prepared = bool(spec.bias or spec.values_from_keys or not spec.qk_norm_weight or spec.qk_norm_after_rotation
-                             or spec.output_gate)
+                             or spec.output_gate or spec.gate_per_head)
         # what only ops.qk_prepare_whole does
         self.whole = bool(spec.qk_norm_whole or spec.rotate_neighbours or spec.value_position is not None)
         if self.whole and (self.prepared or spec.differential is not None or spec.q_temperature is not None or not spec.own_kv):
@@ -92,6 +93,8 @@ class Attention(Mixer):
             raise ValueError("attention: the differential form and the query temperature go with plain projections of its own keys")
         if spec.q_temperature is not None and not (int(spec.q_temperature[1]) > 0):
             raise ValueError("attention: the query temperature's period must be positive")
+        if spec.output_gate and spec.gate_per_head:
+            raise ValueError("attention: the output gate is one per element or one per head")
         if self.general:
             if not self.prepared and not self.whole and (spec.position is not None or spec.qk_norm_eps is not None):
                 raise ValueError("attention: the general form (value width, chunk mask, distance bias) has neither rotation nor q/k norm")
@@ -125,6 +128,7 @@ class Attention(Mixer):
                       "sinks": name("sinks", "sinks"), "lq1": name("lq1", "lambda_q1"), "lk1": name("lk1", "lambda_k1"),
                       "lq2": name("lq2", "lambda_q2"), "lk2": name("lk2", "lambda_k2"), "score_bias": name("score_bias", "score_bias")}
         self.diff_lambda = 0.0
+        self.gate_at = 0                      # the gate's first column in the fused projection
         for role in ("q", "k", "o"):          # a bias is named after its weight unless the specification names it
             weight = self.names[role]
             default = weight[:-len(".weight")] + ".bias" if weight.endswith(".weight") else weight + ".b"
@@ -139,8 +143,8 @@ class Attention(Mixer):
             specs.append(WeightSpec(p + nm["k"], (s.n_kv_heads * self.maps * s.head_dim, s.hidden)))
         if self.own_v:
             specs.append(WeightSpec(p + nm["v"], (s.n_kv_heads * s.value_dim, s.hidden)))
-        if s.output_gate:
-            specs.append(WeightSpec(p + nm["gate"], (s.n_heads * s.value_dim, s.hidden)))
+        if s.output_gate or s.gate_per_head:
+            specs.append(WeightSpec(p + nm["gate"], (s.n_heads * (1 if s.gate_per_head else s.value_dim), s.hidden)))
         specs.append(WeightSpec(p + nm["o"], (s.hidden, s.n_heads * s.value_dim)))
         if s.bias:
             specs.append(WeightSpec(p + nm["q_bias"], (s.n_heads * s.head_dim,), role="vector", init="small"))
@@ -176,8 +180,11 @@ class Attention(Mixer):
             parts.append(tensors[p + nm["k"]])
         if self.own_v:
             parts.append(tensors[p + nm["v"]])
-        if s.output_gate:
+        self.gate_at = sum(t.shape[0] for t in parts)
+        if s.output_gate or s.gate_per_head:
             parts.append(tensors[p + nm["gate"]])
+        if s.gate_per_head and self.prepared:      # a few rows: whole tiles of sixteen for the products (the padding's columns go unread)
+            parts.append(parts[-1].new_zeros(-sum(t.shape[0] for t in parts) % 16, s.hidden))
         self.w_qkv = torch.cat(parts, dim=0).contiguous() if len(parts) > 1 else parts[0]   # rows: q | k | v | gate
         self.w_o = tensors[p + nm["o"]]
         if s.bias:
@@ -220,9 +227,10 @@ class Attention(Mixer):
             qkv = ctx.scratch("attn.qkv", (n, self.w_qkv.shape[0]))
         ops.linear(h, self.w_qkv, qkv)
         o = self._attend_general(ctx, qkv, cache) if self.general else self._attend(ctx, qkv, cache)
-        if s.output_gate:
-            at = self.w_qkv.shape[0] - s.n_heads * s.value_dim
-            ops.sigmoid_gate_strided(o.view(n, s.n_heads * s.value_dim), qkv[:, at:])
+        if s.output_gate or s.gate_per_head:
+            columns = s.n_heads * (1 if s.gate_per_head else s.value_dim)
+            ops.sigmoid_gate_strided(o.view(n, s.n_heads * s.value_dim), qkv[:, self.gate_at:self.gate_at + columns],
+                                     group=s.value_dim if s.gate_per_head else 1)
         out = ctx.scratch("attn.out", (n, s.hidden), torch.float32 if self.output_float32 else None)
         ops.linear(o.view(n, s.n_heads * s.value_dim), self.w_o, out)
         if self.output_bias is not None and not self.defer_output_bias:

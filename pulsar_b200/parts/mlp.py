@@ -1,6 +1,7 @@
 """Dense gated feed-forward."""
 from __future__ import annotations
 
+import math
 from typing import Dict, List
 
 import torch
@@ -14,8 +15,8 @@ from .norm import RMSNorm, accumulate_and_prepare
 
 @FEED_FORWARDS.register("swiglu")
 class SwiGLU(FeedForward):
-    """(silu(h Wg^T) * (h Wu^T)) Wd^T without bias (pulsar-core/src/model/qwen3.cpp:117-119).
-    Gate and up are one fused product (rows: gate | up); the gating runs in float32 and
+    """(act(h Wg^T) * (h Wu^T)) Wd^T without bias (pulsar-core/src/model/qwen3.cpp:117-119), act silu or relu
+    (``spec.activation``).  Gate and up are one fused product (rows: gate | up); the gating runs in float32 and
     rounds once.
 
     Options (``spec.extra``): ``tensor_names`` by role "gate", "up", "down"; ``bias`` True: the three projections have
@@ -27,8 +28,10 @@ class SwiGLU(FeedForward):
     defer_output_bias = False
 
     def __init__(self, spec: FeedForwardSpec, prefix: str, dtype: torch.dtype):
-        if spec.activation != "silu":
-            raise ValueError(f"swiglu: activation '{spec.activation}' is not implemented (only 'silu')")
+        if spec.activation not in ("silu", "relu"):
+            raise ValueError(f"swiglu: activation '{spec.activation}' is not implemented (only 'silu' and 'relu')")
+        # relu is the gating's limit of a steep sigmoid: no clamp, alpha infinite, nothing added to the up part
+        self.gating = None if spec.activation == "silu" else (math.inf, math.inf, 0.0)
         self.spec, self.prefix, self.dtype = spec, prefix, dtype
         names = dict(spec.option("tensor_names", ()))
         self.names = {r: names.get(r, d) for r, d in (("gate", "gate_proj.weight"), ("up", "up_proj.weight"),
@@ -70,9 +73,9 @@ class SwiGLU(FeedForward):
         if not (ops.fused_projection_supported(n, self.w_gate_up, swiglu=True) and ops.fused_projection_supported(n, self.w_down)):
             return False
         act = ctx.scratch("mlp.act", (n, s.intermediate))
-        prepared = ctx.prepared_norms.pop(id(norm), None) if ops.FUSED_NORM_MLP else None
+        prepared = ctx.prepared_norms.pop(id(norm), None) if ops.FUSED_NORM_MLP and self.gating is None else None
         if prepared is None or not ops.linear_prenormed(prepared[0], prepared[1], norm.spec.eps, self.w_gate_up, act, swiglu=True):
-            ops.gated_linear(ctx, norm.forward(ctx, residual, None), self.w_gate_up, act)
+            ops.gated_linear(ctx, norm.forward(ctx, residual, None), self.w_gate_up, act, gating=self.gating)
         ctx.prepared_norms.clear()              # the residual changes now
         if not accumulate_and_prepare(ctx, act, self.w_down, residual, next_norm):
             raise ops.KernelError("swiglu: the down projection refused sizes it had declared supported")
@@ -85,9 +88,9 @@ class SwiGLU(FeedForward):
             # float32 rows of the product, the biases added before anything is rounded
             gate_up = ctx.scratch("mlp.gate_up32", (n, 2 * s.intermediate), torch.float32)
             ops.linear(h, self.w_gate_up, gate_up)
-            ops.glu_bias(gate_up, self.b_gate_up, act)
+            ops.glu_bias(gate_up, self.b_gate_up, act, self.gating)
         else:
-            ops.gated_linear(ctx, h, self.w_gate_up, act)
+            ops.gated_linear(ctx, h, self.w_gate_up, act, gating=self.gating)
         out = ctx.scratch("mlp.out", (n, s.hidden))
         ops.linear(act, self.w_down, out)
         if self.output_bias is not None and not self.defer_output_bias:

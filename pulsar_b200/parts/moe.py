@@ -28,13 +28,16 @@ class MixtureOfExperts(FeedForward):
     With ``scoring`` "softmax" the scores are s = softmax(W_r h) over all experts instead of sigmoids, and ``renorm_eps`` is added
     to the chosen scores' sum before a renormalising division.
 
+    With ``router_bias`` (a tensor name behind the prefix, one number per router output) the logits are W_r h + bias.  With
+    ``scoring`` "softmax", ``renormalize`` and no ``renorm_eps`` the weights are the softmax over the chosen logits alone.
+
     With ``gated`` False an expert is W_down max(W_up h, 0)^2 (``spec.activation`` "relu2"; no gate projection).  ``identity`` more
     outputs of the router stand for experts that return their input and have no tensors.  ``correction`` (a tensor name behind
     the prefix, one number per router output) joins the scores for the choice, not for the weights.  ``groups`` = (count, keep):
     the router's outputs form ``count`` groups of neighbours, a group counts as its best choice score, and the chosen come from
     the ``keep`` best groups.
 
-    Options (``spec.extra``): ``experts``, ``top``, ``router_scale``, ``renormalize``, ``scoring``, ``renorm_eps``, ``limit``, ``alpha``, ``shift``,
+    Options (``spec.extra``): ``experts``, ``top``, ``router_scale``, ``renormalize``, ``scoring``, ``renorm_eps``, ``router_bias``, ``limit``, ``alpha``, ``shift``,
     ``gated``, ``identity``, ``correction``, ``groups``, ``weight_input``, ``shared`` (FeedForwardSpec or None), ``shared_prefix`` ("shared."), ``shared_gate``, ``tensor_names``
     by role "router", "gate", "up", "down" (an expert's tensors are ``<prefix>e<i>.<name>``).
 
@@ -75,6 +78,8 @@ class MixtureOfExperts(FeedForward):
             raise ValueError("moe: weights on the experts' inputs go with gated experts and no identity experts")
         self.correction_name = prefix + str(spec.option("correction")) if spec.option("correction", None) else None
         self.correction = None
+        self.router_bias_name = prefix + str(spec.option("router_bias")) if spec.option("router_bias", None) else None
+        self.router_bias = None
         shared = spec.option("shared", None)
         self.shared = self.shared_gate_name = None
         if shared is not None:
@@ -97,6 +102,8 @@ class MixtureOfExperts(FeedForward):
         specs.append(WeightSpec(self.prefix + self.names["router"], (self.outputs, s.hidden), role="vector", init="normal"))
         if self.correction_name is not None:
             specs.append(WeightSpec(self.correction_name, (self.outputs,), role="vector", init="small"))
+        if self.router_bias_name is not None:
+            specs.append(WeightSpec(self.router_bias_name, (self.outputs,), role="vector", init="small"))
         if self.shared is not None:
             specs += self.shared.weight_specs()
         if self.shared_gate_name is not None:
@@ -112,6 +119,8 @@ class MixtureOfExperts(FeedForward):
             self.w_gate_up = torch.stack([tensors[self._expert(i, "up")] for i in range(n)]).contiguous()       # [E, ff, width]
         if self.correction_name is not None:
             self.correction = tensors[self.correction_name].contiguous()
+        if self.router_bias_name is not None:
+            self.router_bias = tensors[self.router_bias_name].contiguous()
         self.w_down = torch.stack([tensors[self._expert(i, "down")] for i in range(n)]).contiguous()    # [E, width, ff]
         self.router = tensors[self.prefix + self.names["router"]].contiguous()
         if self.shared_gate_name is not None:           # one more row of the router's product: it competes for nothing
@@ -131,7 +140,8 @@ class MixtureOfExperts(FeedForward):
         weights = ctx.scratch("moe.weights", (n, top), torch.float32)
         shared_scale = ctx.scratch("moe.shared_scale", (n, 1), torch.float32) if self.shared_gate_name is not None else None
         ops.moe_route(h, self.router, ids, weights, self.router_scale, self.renormalize, shared_scale,
-                      softmax=self.scoring == "softmax", renorm_eps=self.renorm_eps, correction=self.correction, groups=self.groups)
+                      softmax=self.scoring == "softmax", renorm_eps=self.renorm_eps, correction=self.correction, groups=self.groups,
+                      logit_bias=self.router_bias)
         shared = self.shared.forward(ctx, h) if self.shared is not None else None
         act = ctx.scratch("moe.act", (n * top, s.intermediate))
         out = ctx.scratch("moe.out", (n, s.hidden))
