@@ -116,15 +116,16 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor) -> torc
 
 
 def scalar_decay_scan(x, B, C, dt, rate, skip):
-    """x [L, H, V], B and C [L, H, N], dt [L, H], rate and skip [H] -> [L, H, V], token by token: a head's state decays by
-    exp(-rate * dt) as a whole."""
+    """x [L, H, V], B and C [L, H, N], dt [L, H], rate and skip [H] -> (y [L, H, V], spread [L, H, V]), token by token: a head's
+    state decays by exp(-rate * dt) as a whole.  ``spread`` is y with the magnitude of every term in its place."""
     L, H, V = x.shape
     S = x.new_zeros(H, B.shape[2], V)
-    out = x.new_zeros(L, H, V)
+    out, spread = x.new_zeros(L, H, V), x.new_zeros(L, H, V)
     for t in range(L):
         S = torch.exp(-rate * dt[t])[:, None, None] * S + dt[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :]
         out[t] = torch.einsum("hnv,hn->hv", S, C[t]) + skip[:, None] * x[t]
-    return out
+        spread[t] = torch.einsum("hnv,hn->hv", S.abs(), C[t].abs()) + (skip[:, None] * x[t]).abs()
+    return out, spread
 
 
 def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
@@ -133,7 +134,8 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, par
     return rms_norm(y.view(y.shape[0], parts, -1), None, eps).reshape(y.shape) * weight
 
 
-def mamba2(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
+def mamba2(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float, cancellations: Optional[list] = None) -> torch.Tensor:
+    """``cancellations`` receives, per token, how much is left of a normed part after cancellation (the least over the parts)."""
     L = h.shape[0]
     H, V, N, G = int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"])
     inner = H * V
@@ -143,14 +145,18 @@ def mamba2(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> 
     x, B, C = torch.split(xbc, [inner, G * N, G * N], dim=-1)
     B, C = (t.view(L, G, N).repeat_interleave(H // G, dim=1) for t in (B, C))
     dt = torch.nn.functional.softplus(dt + w["dt_bias"], threshold=1e9)
-    y = scalar_decay_scan(x.view(L, H, V), B, C, dt, torch.exp(w["A_log"]), w["D"]).reshape(L, inner)
-    return gated_group_norm(y, z, w["norm"], int(m["norm_groups"]), eps) @ w["o"].T
+    y, spread = (t.reshape(L, inner) for t in scalar_decay_scan(x.view(L, H, V), B, C, dt, torch.exp(w["A_log"]), w["D"]))
+    parts = int(m["norm_groups"])
+    if cancellations is not None:
+        size = lambda t: ((t * z * torch.sigmoid(z)).view(L, parts, -1) ** 2).mean(-1).sqrt()
+        cancellations.append((size(y) / size(spread).clamp_min(1e-30)).min(dim=-1).values)
+    return gated_group_norm(y, z, w["norm"], parts, eps) @ w["o"].T
 
 
-def side_by_side(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
+def side_by_side(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float, cancellations: Optional[list] = None) -> torch.Tensor:
     """Half the sum of the two outputs, each normed over the width with a weight of its own."""
     left = rms_norm(window_attention(h, sub(w, "left."), m["left"]), w["left.out"], eps)
-    right = rms_norm(mamba2(h, sub(w, "right."), m["right"], eps), w["right.out"], eps)
+    right = rms_norm(mamba2(h, sub(w, "right."), m["right"], eps, cancellations), w["right.out"], eps)
     return 0.5 * (left + right)
 
 
@@ -200,7 +206,7 @@ def layer(x: torch.Tensor, w: Dict[str, torch.Tensor], spec: dict, eps: float, m
           cancellations: Optional[list] = None) -> torch.Tensor:
     h = rms_norm(x, w["norm1"], eps)
     if spec["type"] == "parallel":
-        x = x + side_by_side(h, sub(w, "mix."), spec["mixer"], eps)
+        x = x + side_by_side(h, sub(w, "mix."), spec["mixer"], eps, cancellations)
     else:
         x = x + mlstm(h, sub(w, "mix."), spec["mixer"], eps, cancellations)
     mlp = spec.get("mlp")
@@ -214,8 +220,8 @@ def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: List[int], dtyp
             streams: Optional[list] = None, margins: Optional[list] = None, cancellations: Optional[list] = None) -> torch.Tensor:
     """Logits [L, vocab] of one whole sequence.  ``streams`` receives the stream after every layer; ``margins`` receives
     per-token margins of every routed layer (``route_margins``: a small one marks a token at which rounding to 16 bits may choose
-    other experts), ``cancellations`` what cancellation leaves of every matrix memory's output (``matrix_memory``: a small one
-    marks a token at which rounding is magnified)."""
+    other experts), ``cancellations`` what cancellation leaves of every recurrence's output before it is normed (``matrix_memory``,
+    ``mamba2``: a small one marks a token at which rounding is magnified)."""
     w = {n: t.to(dtype) for n, t in weights.items()}
     eps = float(cfg["norm"]["eps"])
     x = w["embed"][torch.tensor(list(tokens))] * float((cfg.get("embedding") or {}).get("scale", 1.0))
