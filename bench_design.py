@@ -2,7 +2,7 @@
 
 For each size the design's model and a Qwen3 dense model of the same width, depth, heads, feed-forward size and vocabulary
 (for Megusun and Bumotar: a Topunex model, the closest one, with the same width, depth, projection sizes, experts and vocabulary;
-its entry keeps the key "dense"; for Rikolix two models: Topunex with feed-forwards of equal numbers of weights, and under
+its entry keeps the key "dense", as does Bumotar's for Bosenex; for Rikolix two models: Topunex with feed-forwards of equal numbers of weights, and under
 "latent" Bumotar for the layers with a latent) are built with random weights (bfloat16) and timed through the step function:
 
   prefill   one step of 2,048 prompt tokens (tokens a second, ms)
@@ -212,6 +212,7 @@ def bumotar_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
         "moe_gate_up": (L * (n * top * 2 * fe * w * 2 + n * w * 2), L * 4.0 * n * top * fe * w, "fp32 FMA"),
         "moe_down": (L * (n * top * fe * w * 2 + n * w * 4), L * 2.0 * n * top * fe * w, "fp32 FMA"),
         "silu_mul": (L * n * fs * 6, 0.0, ""),
+        "gemm_tcgen05": (L * (2 * fs * w + n * (w + fs)) * 2, L * 2.0 * n * w * 2 * fs, "bf16 tensor"),       # the shared experts' gated products
     }
     return {k: (b * steps, f * steps, on) for k, (b, f, on) in work.items()}
 
@@ -321,6 +322,77 @@ def rikolix_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
         "moe_down": (Lm * (n * real * fe * w * 2 + n * w * 4), Lm * 2.0 * n * real * fe * w, "fp32 FMA"),
     }
     return {k: (b * steps, f * steps, on) for k, (b, f, on) in work.items()}
+
+
+# Bosenex at sizes that resemble layers of real models: of every four layers one has a window attention (heads of 128, half of each
+# rotating, a cap, a window of 1,024) beside a state space (twice the width in heads of 64, states of 128 in two groups, a convolution
+# of 4 taps), three have a matrix memory (as many heads, keys of 64, values of 128); two layers have dense ReLU-gated feed-forwards,
+# six have 32 clamped experts of which a token uses 4, beside a shared expert.  The shape also carries what the model beside it
+# needs (Bumotar: eight layer runs, five of them a window attention beside a retention of the same heads, three with a latent).
+BOSENEX_SIZES = {name: dict(z, ssm_heads=2 * z["width"] // 64, ssm_vdim=64, ssm_state=128, ssm_groups=2, conv=4)
+                 for name, z in BUMOTAR_SIZES.items()}
+BOSENEX_LAYERS = [("parallel", "moe"), ("memory", "moe"), ("memory", "dense"), ("memory", "moe")] * 2
+
+
+def bosenex_config(z: dict) -> dict:
+    left = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["dim"], scale=1.0 / math.sqrt(z["dim"]), softcap=30.0,
+                mask=dict(size=z["window"]), rot=dict(base=100000.0, dims=z["rot"]))
+    right = dict(heads=z["ssm_heads"], vdim=z["ssm_vdim"], state=z["ssm_state"], groups=z["ssm_groups"], conv=z["conv"],
+                 norm_groups=z["ssm_groups"])
+    memory = dict(heads=z["heads"], dim=z["ret_dim"], vdim=z["ret_vdim"], gate_cap=12.0)
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"], limit=7.0), router=dict(experts=z["experts"], top=z["top"]),
+               shared=dict(ff=z["shared_ff"], limit=7.0))
+    layers = [dict(type="parallel" if mixer == "parallel" else "mlstm", mixer=dict(left=dict(left), right=dict(right)) if mixer == "parallel" else dict(memory),
+                   mlp=dict(kind="dense", ff=z["ff"]) if ff == "dense" else dict(moe)) for mixer, ff in BOSENEX_LAYERS]
+    return dict(architecture="Bosenex", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), embedding=dict(scale=1.0), layers=layers)
+
+
+def bosenex_work(z: dict, phase: str) -> Dict[str, Tuple[float, float, str]]:
+    """Per kernel class of Bosenex: (bytes it must move, flops, what the flops run on) summed over the layers of a step."""
+    n = PROMPT if phase == "prefill" else BATCH
+    seqs = 1 if phase == "prefill" else BATCH
+    start = 0 if phase == "prefill" else CONTEXT - 1
+    Lp, Lm = (sum(1 for m, _ in BOSENEX_LAYERS if m == k) for k in ("parallel", "memory"))
+    Ld, Le = (sum(1 for _, f in BOSENEX_LAYERS if f == k) for k in ("dense", "moe"))
+    L, w, H, G, d = Lp + Lm, z["width"], z["heads"], z["kv_heads"], z["dim"]
+    D, V = z["ret_dim"], z["ret_vdim"]
+    E, top, fe, fs = z["experts"], z["top"], z["expert_ff"], z["shared_ff"]
+    steps = 1 if phase == "prefill" else 4
+    win_pairs = seqs * _window_pairs(n // seqs, start, z["window"], 0)
+    keys_read = seqs * min(start + n // seqs, z["window"] + (n // seqs if phase == "prefill" else 0))
+    attention = (Lp * (keys_read * G * 2 * d * 2 + n * H * d * (4 + 2)), Lp * 4.0 * H * d * win_pairs)
+    # a recurrence reads its rows once and writes its output, reads and writes the kept states, and in chunks of 64 tokens writes a
+    # state per chunk and head, folds it and reads it; operations: state and query products, and the scores within a chunk
+    chunk = 64
+    chunks = n // chunk if phase == "prefill" else 0
+    memory = (Lm * (n * ((2 * H * (D + V) + 2 * H) * 4 + H * V * 2) + seqs * H * D * V * 8 + chunks * H * D * V * 4 * 3),
+              Lm * n * H * (4.0 * D * V + (chunk * (D + V) if phase == "prefill" else 0.0)))
+    Hs, Vs, N, Gs = z["ssm_heads"], z["ssm_vdim"], z["ssm_state"], z["ssm_groups"]
+    ch = Hs * Vs + 2 * Gs * N
+    space = (Lp * (n * ((Hs * Vs + ch + Hs) * 4 + Hs * Vs * 2) + seqs * (Hs * N * Vs + ch * (z["conv"] - 1)) * 8 + chunks * Hs * N * Vs * 4 * 3),
+             Lp * n * Hs * (4.0 * N * Vs + (chunk * (N + Vs) if phase == "prefill" else 0.0)))
+    on = "bf16 tensor" if phase == "prefill" else "fp32 FMA"
+    distinct = E * (1.0 - (1.0 - top / E) ** n)
+    work = {
+        "paged_attention_general_tc": (attention[0], attention[1], "bf16 tensor"),
+        "paged_attention_general_tiled": (attention[0], attention[1], "fp32 FMA"),
+        "paged_attention_general": (attention[0], attention[1], "fp32 FMA"),
+        "matrix_memory": (memory[0], memory[1], on),
+        "state_space": (space[0], space[1], on),
+        "causal_conv_silu": (Lp * n * ch * (4 + 2), 0.0, ""),
+        "qk_prepare": (Lp * n * ((H + 2 * G) * d * 4 + H * d * 4 + 2 * G * d * 2), 0.0, ""),
+        "sigmoid_gate_strided": (Lp * n * H * (d * 4 + 4), 0.0, ""),
+        "normed_sum": (Lp * n * w * (4 + 4 + 2), 0.0, ""),
+        "add_rmsnorm": ((2 * L + 1) * n * w * (4 + 4 + 2 + 2), 0.0, ""),
+        "moe_route": (Le * (n * w * 2 + E * w * 4), 0.0, ""),
+        "moe_grouped": (Le * (distinct * 3 * w * fe * 2 + n * w * 4 + n * top * (fe * 4 + w * 8)), Le * 2.0 * n * top * 3 * w * fe, "bf16 tensor"),
+        "moe_gate_up": (Le * (n * top * 2 * fe * w * 2 + n * w * 2), Le * 4.0 * n * top * fe * w, "fp32 FMA"),
+        "moe_down": (Le * (n * top * fe * w * 2 + n * w * 4), Le * 2.0 * n * top * fe * w, "fp32 FMA"),
+        # the gated products of the dense and the shared feed-forwards
+        "gemm_tcgen05": (Ld * (2 * z["ff"] * w + n * (w + z["ff"])) * 2 + Le * (2 * fs * w + n * (w + fs)) * 2,
+                         2.0 * n * w * 2 * (Ld * z["ff"] + Le * fs), "bf16 tensor"),
+    }
+    return {k: (b * steps, f * steps, on_) for k, (b, f, on_) in work.items()}
 
 
 def dense_config(z: dict) -> dict:
@@ -530,7 +602,8 @@ DESIGNS = {"bubotar": (SIZES, bubotar_config, own_work, dense_config, like_work)
            "megusun": (MEGUSUN_SIZES, megusun_config, megusun_work, topunex_config, topunex_work),
            "bumotar": (BUMOTAR_SIZES, bumotar_config, bumotar_work, topunex_config, topunex_work),
            "rikolix": (RIKOLIX_SIZES, rikolix_config, rikolix_work, rikolix_topunex_config, rikolix_topunex_work,
-                       rikolix_bumotar_config, rikolix_bumotar_work)}
+                       rikolix_bumotar_config, rikolix_bumotar_work),
+           "bosenex": (BOSENEX_SIZES, bosenex_config, bosenex_work, bumotar_config, bumotar_work)}
 
 
 def run(args, bench) -> dict:
@@ -545,7 +618,7 @@ def run(args, bench) -> dict:
     for size in sizes:
         z = table[size]
         entry = {"shape": z}
-        # "dense": the model beside it (Qwen3 dense, or Topunex for Megusun, Bumotar and Rikolix)
+        # "dense": the model beside it (Qwen3 dense, or Topunex for Megusun, Bumotar and Rikolix, or Bumotar for Bosenex)
         models = [("design", make_config(z), design_work), ("dense", beside_config(z), beside_work)]
         if second:
             models.append(("latent", second[0](z), second[1]))
