@@ -23,7 +23,7 @@
 //                            fold    S_in(c) = state entering chunk c; S <- decay(c) S + U_c along a sequence  (per element)
 //                            out     r_i = sum_(j<=i) decay(j..i) b_j (q_i . k_j) v_j + decay(..i) S_in^T q_i
 //                          q, k and v are rounded to bfloat16 once (as projections may be); everything of the recurrence
-//                          that meets a tensor core (weighted keys, weighted scores, the entering state) is split into two
+//                          that meets a tensor core (weighted values, weighted scores, the entering state) is split into two
 //                          bfloat16 numbers, hi + lo (16 bits of mantissa together), and enters two MMAs with the same
 //                          float32 accumulator.  The normaliser n and its products are float32 on CUDA cores.
 //   gates, gated_norm      what stands before the chunks (log decays and input weights per token and head; for the matrix memory
@@ -228,23 +228,32 @@ __global__ void __launch_bounds__(THREADS) recurrence_step_kernel(const StepArgs
 // ------------------------------------------------------------------------------------------------ gates
 // Log decays, input weights and floors of the matrix memory, [N, H]: a block per (head, sequence) walks the tokens blockDim at a
 // time.  A token maps m to max(f + m, i); maps compose as (F, M) then (f, i) = (F + f, max(f + M, i)), so the block scans them.
-__global__ void __launch_bounds__(512) memory_gates_kernel(const float* __restrict__ rows, long stride, int i_off, int f_off, const float* __restrict__ i_bias,
+__global__ void __launch_bounds__(1024) memory_gates_kernel(const float* __restrict__ rows, long stride, int i_off, int f_off, const float* __restrict__ i_bias,
                                     const float* __restrict__ f_bias, float cap, const Step st, long m_off, int H,
                                     float* __restrict__ ld, float* __restrict__ wt, float* __restrict__ floor_out) {
     pdl_wait();
-    __shared__ float wf[16], wm[16], last;
+    __shared__ float wf[32], wm[32], last;
     const int h = blockIdx.x, s = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int t0 = st.cu_q[s], t1 = st.cu_q[s + 1];
     float* kept_m = st.state + (size_t)st.state_slots[s] * st.state_stride + m_off + h;
     float m_in = *kept_m;
     const float bi = i_bias[h], bf = f_bias[h];
+    float pre_i = 0.0f, pre_f = 0.0f;                     // the next round's pre-activations, fetched a round ahead
+    if (t0 + (int)threadIdx.x < t1) {
+        pre_i = rows[(size_t)(t0 + threadIdx.x) * stride + i_off + h];
+        pre_f = rows[(size_t)(t0 + threadIdx.x) * stride + f_off + h];
+    }
     for (int base = t0; base < t1; base += blockDim.x) {
         const int t = base + threadIdx.x;
         const bool in = t < t1;
         float gi = -INFINITY, gf = 0.0f;                  // behind the end: a map that changes nothing
         if (in) {
-            gi = capped(rows[(size_t)t * stride + i_off + h] + bi, cap);
-            gf = log_sigmoid_f(capped(rows[(size_t)t * stride + f_off + h] + bf, cap));
+            gi = capped(pre_i + bi, cap);
+            gf = log_sigmoid_f(capped(pre_f + bf, cap));
+        }
+        if (t + (int)blockDim.x < t1) {
+            pre_i = rows[(size_t)(t + blockDim.x) * stride + i_off + h];
+            pre_f = rows[(size_t)(t + blockDim.x) * stride + f_off + h];
         }
         float F = gf, M = gi;
 #pragma unroll
@@ -308,27 +317,41 @@ template <typename T> struct Source {
     int share;
 };
 
+// A chunk's state of a head in memory: [D, V] filled up to whole tiles of 16 rows and 8 columns (Dp, Vp; zeros), tile by tile
+// (rows of tiles first) in the order in which the lanes of a warp take a B operand of m16n8k16: lane l holds column l / 4 and
+// rows 2 (l % 4), 2 (l % 4) + 1 and the same + 8, four numbers of 16 bytes.  The normaliser's D numbers follow.
 struct ChunkShape {
     const int* cu_q;
     int n_seqs, H, D, V, normaliser;
-    long per;                // floats of U per (chunk, head): D * V, then D for the normaliser, rounded up to a multiple of four
+    int Dp, Vp;
+    long per;                // words of U per (chunk, head): Dp * Vp, then D for the normaliser, rounded up to a multiple of four
     float q_scale;
+    int heads;               // heads of a block; they read the same q and k
 };
 
-// cum[j] = sum of the chunk's log decays up to and including token j (warp 0; two tokens a lane), zero log decay behind the end.
-__device__ __forceinline__ void cumulative_decays(const float* __restrict__ ld, int H, int h, int t0, int n, float* cum) {
-    if (threadIdx.x >= 32) return;
+// What warp 0 leaves for a head: cum[j], the sum of the chunk's log decays up to and including token j (zero log decay behind the end;
+// two tokens a lane), and weight[j] = the token's input weight, times (kBehind) the decay behind it.  Returns the whole sum.
+template <bool kBehind>
+__device__ __forceinline__ float chunk_decays(const float* __restrict__ ld, const float* __restrict__ wt, int H, int h, int t0, int n, float* cum,
+                                              float* weight) {
     const int lane = threadIdx.x, j = 2 * lane;
-    const float a = j < n ? fmaxf(ld[(size_t)(t0 + j) * H + h], kLeastLogDecay) : 0.0f;
-    const float b = j + 1 < n ? fmaxf(ld[(size_t)(t0 + j + 1) * H + h], kLeastLogDecay) : 0.0f;
+    const bool in_a = j < n, in_b = j + 1 < n;
+    const size_t at = (size_t)(t0 + j) * H + h;
+    const float a = in_a ? fmaxf(ld[at], kLeastLogDecay) : 0.0f, b = in_b ? fmaxf(ld[at + H], kLeastLogDecay) : 0.0f;
+    float wa = in_a ? wt[at] : 0.0f, wb = in_b ? wt[at + H] : 0.0f;
     float sum = a + b;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
         const float p = __shfl_up_sync(0xffffffffu, sum, o);
         if (lane >= o) sum += p;
     }
+    const float all = __shfl_sync(0xffffffffu, sum, 31);
+    if (kBehind) { wa *= expf(all - (sum - b)); wb *= expf(all - sum); }
     cum[j] = sum - b;
     cum[j + 1] = sum;
+    weight[j] = wa;
+    weight[j + 1] = wb;
+    return all;
 }
 
 template <typename T> __device__ __forceinline__ void load4(const T* src, bool vec, int left, float (&v)[4]) {
@@ -340,16 +363,57 @@ template <typename T> __device__ __forceinline__ void load4(const T* src, bool v
     }
 }
 
-// Element columns [c0, c0 + width) of n rows -> shared rows of bfloat16 (stride `ld_s`); zeros behind `limit` columns and n rows.
+template <typename T> __device__ __forceinline__ bool quads_aligned(const T* src, long tok, int limit) {
+    return (limit & 3) == 0 && (((uintptr_t)src | (uintptr_t)(tok * (long)sizeof(T))) & (4 * sizeof(T) - 1)) == 0;
+}
+
+// How 128 threads walk rows of `parts` vectors: a power of two of neighbouring threads per row, the rest over the rows.
+struct Lanes {
+    int lanes, lane, row, rows;
+    __device__ __forceinline__ explicit Lanes(int parts) {
+        const int bits = parts >= 128 ? 7 : parts <= 1 ? 0 : 32 - __clz(parts - 1);
+        lanes = 1 << bits;
+        lane = threadIdx.x & (lanes - 1);
+        row = threadIdx.x >> bits;
+        rows = 128 >> bits;
+    }
+};
+
+// Columns [0, limit) of n rows -> kChunk shared rows of bfloat16, `width` columns (stride ld_s); zeros behind the limit and the n rows.
 template <typename T>
 __device__ __forceinline__ void stage_rows(const T* __restrict__ src, long tok, int n, int limit, int width, bf16* dst, int ld_s) {
-    const int quads = width >> 2;
-    const bool vec = (limit & 3) == 0 && (((uintptr_t)src | (uintptr_t)(tok * (long)sizeof(T))) & (4 * sizeof(T) - 1)) == 0;
-    for (int i = threadIdx.x; i < kChunk * quads; i += blockDim.x) {
-        const int j = i / quads, d = (i - j * quads) << 2;
-        float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        if (j < n && d < limit) load4(src + (size_t)j * tok + d, vec, limit - d, v);
-        store_quad(dst + j * ld_s + d, v);
+    if (sizeof(T) == 2 && (limit & 7) == 0 && (((uintptr_t)src | (uintptr_t)(tok * 2)) & 15) == 0) {      // bfloat16 rows as they are
+        const Lanes at(width >> 3);
+        for (int d = at.lane << 3; d < width; d += at.lanes << 3)
+#pragma unroll 8
+            for (int j = at.row; j < kChunk; j += at.rows) {
+                const bool in = j < n && d < limit;
+                cp_async16(smem_u32(dst + j * ld_s + d), in ? src + (size_t)j * tok + d : src, in);
+            }
+        cp_async_commit();
+        cp_async_wait<0>();
+        return;
+    }
+    const Lanes at(width >> 2);
+    const bool vec = quads_aligned(src, tok, limit);
+    for (int d = at.lane << 2; d < width; d += at.lanes << 2) {
+        if (vec && n == kChunk && d < limit) {            // whole rows: the loads of eight of them in flight together
+            for (int j0 = at.row; j0 < kChunk; j0 += 8 * at.rows) {
+                float v[8][4];
+#pragma unroll
+                for (int k = 0; k < 8; ++k)
+                    if (j0 + k * at.rows < kChunk) load_quad(src + (size_t)(j0 + k * at.rows) * tok + d, v[k]);
+#pragma unroll
+                for (int k = 0; k < 8; ++k)
+                    if (j0 + k * at.rows < kChunk) store_quad(dst + (j0 + k * at.rows) * ld_s + d, v[k]);
+            }
+            continue;
+        }
+        for (int j = at.row; j < kChunk; j += at.rows) {
+            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            if (j < n && d < limit) load4(src + (size_t)j * tok + d, vec, limit - d, v);
+            store_quad(dst + j * ld_s + d, v);
+        }
     }
 }
 
@@ -359,274 +423,292 @@ __global__ void __launch_bounds__(128) recurrence_chunk_state_kernel(const Sourc
     pdl_wait();
     extern __shared__ __align__(16) unsigned char raw_smem[];
     __shared__ float cum[kChunk], coef[kChunk];
-    const int Dp = (sh.D + 15) & ~15, ldk = Dp + kPad, ldv = kCols + kPad;
-    bf16* kh = reinterpret_cast<bf16*>(raw_smem);         // [kChunk][ldk] weighted keys, high halves
-    bf16* kl = kh + kChunk * ldk;                         // low halves
-    bf16* vs = kl + kChunk * ldk;                         // [kChunk][ldv]
-    const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kCols;
+    const int ldk = sh.Dp + kPad, ldv = kCols + kPad;
+    bf16* ks = reinterpret_cast<bf16*>(raw_smem);         // [kChunk][ldk]
+    bf16* vh = ks + kChunk * ldk;                         // [kChunk][ldv] weighted values, high halves
+    bf16* vl = vh + kChunk * ldv;                         // low halves
+    const int chunk = blockIdx.x, h0 = blockIdx.y * sh.heads, v0 = blockIdx.z * kCols;
     int s, t0, t1;
     if (!find_chunk(sh.cu_q, sh.n_seqs, chunk, s, t0, t1)) return;
-    const int n = t1 - t0;
-    cumulative_decays(ld, sh.H, h, t0, n, cum);
-    __syncthreads();
-    for (int j = threadIdx.x; j < kChunk; j += blockDim.x)
-        coef[j] = j < n ? expf(cum[kChunk - 1] - cum[j]) * wt[(size_t)(t0 + j) * sh.H + h] : 0.0f;
-    if (threadIdx.x == 0 && v0 == 0) total[(size_t)chunk * sh.H + h] = cum[kChunk - 1];
-    __syncthreads();
-    {
-        const T* src = in.k + (size_t)t0 * in.tok + (size_t)(h / in.share) * sh.D;
-        const int quads = Dp >> 2;
-        const bool vec = (sh.D & 3) == 0 && (((uintptr_t)src | (uintptr_t)(in.tok * (long)sizeof(T))) & (4 * sizeof(T) - 1)) == 0;
-        for (int i = threadIdx.x; i < kChunk * quads; i += blockDim.x) {
-            const int j = i / quads, d = (i - j * quads) << 2;
-            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            if (j < n && d < sh.D) load4(src + (size_t)j * in.tok + d, vec, sh.D - d, v);
-            const float w = coef[j];
-            uint2 hi, lo;
-            split_bf16(v[0] * w, v[1] * w, hi.x, lo.x);
-            split_bf16(v[2] * w, v[3] * w, hi.y, lo.y);
-            *reinterpret_cast<uint2*>(kh + j * ldk + d) = hi;
-            *reinterpret_cast<uint2*>(kl + j * ldk + d) = lo;
-        }
-    }
-    stage_rows(in.v + (size_t)t0 * in.tok + (size_t)h * sh.V + v0, in.tok, n, min(sh.V - v0, kCols), kCols, vs, ldv);
-    __syncthreads();
-    float* out = U + ((size_t)chunk * sh.H + h) * sh.per;
-    if (sh.normaliser && v0 == 0)
-        for (int d = threadIdx.x; d < sh.D; d += blockDim.x) {
-            float sum = 0.0f;
-            for (int j = 0; j < n; ++j) sum += __bfloat162float(kh[j * ldk + d]) + __bfloat162float(kl[j * ldk + d]);
-            out[(size_t)sh.D * sh.V + d] = sum;
-        }
+    const int n = t1 - t0, cols = min(sh.V - v0, kCols);
+    const int NT = sh.Vp >> 3, nt0 = v0 >> 3, tiles = min(NT - nt0, kCols / 8);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tq = lane & 3;
     const int k_steps = (n + 15) >> 4;
-    const int v_tiles = (min(sh.V - v0, kCols) + 15) >> 4;          // pairs of eight columns
-    for (int mt = warp; mt < Dp / 16; mt += 4) {
-        float acc[kCols / 8][4];
+    stage_rows(in.k + (size_t)t0 * in.tok + (size_t)(h0 / in.share) * sh.D, in.tok, n, sh.D, sh.Dp, ks, ldk);
+    for (int h = h0; h < h0 + sh.heads; ++h) {
+        __syncthreads();                                  // the head before has been read
+        if (warp == 0) {
+            const float all = chunk_decays<true>(ld, wt, sh.H, h, t0, n, cum, coef);
+            if (lane == 0 && v0 == 0) total[(size_t)chunk * sh.H + h] = all;
+        }
+        __syncthreads();
+        {
+            const T* src = in.v + (size_t)t0 * in.tok + (size_t)h * sh.V + v0;
+            const bool vec = quads_aligned(src, in.tok, cols);
+            const int v = (threadIdx.x & (kCols / 4 - 1)) << 2, row = threadIdx.x / (kCols / 4);
+            constexpr int kRows = 128 / (kCols / 4);
+            float xs[kChunk / kRows][4];
 #pragma unroll
-        for (int i = 0; i < kCols / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
-        for (int ks = 0; ks < k_steps; ++ks) {
-            const int j = ks * 16 + (lane & 7) + ((lane >> 4) << 3), d = mt * 16 + ((lane >> 3) & 1) * 8;
-            uint32_t ah[4], al[4];
-            ldmatrix_x4_trans(ah, smem_u32(kh + j * ldk + d));
-            ldmatrix_x4_trans(al, smem_u32(kl + j * ldk + d));
-            const int vr = ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
+            for (int k = 0; k < kChunk / kRows; ++k) {
+                xs[k][0] = xs[k][1] = xs[k][2] = xs[k][3] = 0.0f;
+                if (row + k * kRows < n && v < cols) load4(src + (size_t)(row + k * kRows) * in.tok + v, vec, cols - v, xs[k]);
+            }
 #pragma unroll
-            for (int i = 0; i < kCols / 16; ++i) {
-                if (i < v_tiles) {
-                    uint32_t b[4];
-                    ldmatrix_x4_trans(b, smem_u32(vs + vr * ldv + i * 16 + (lane >> 4) * 8));
-                    mma_bf16(acc[2 * i], ah, b[0], b[1]);
-                    mma_bf16(acc[2 * i + 1], ah, b[2], b[3]);
-                    mma_bf16(acc[2 * i], al, b[0], b[1]);
-                    mma_bf16(acc[2 * i + 1], al, b[2], b[3]);
-                }
+            for (int k = 0; k < kChunk / kRows; ++k) {
+                const int j = row + k * kRows;
+                const float (&x)[4] = xs[k];
+                const float w = coef[j];
+                uint2 hi, lo;
+                split_bf16(x[0] * w, x[1] * w, hi.x, lo.x);
+                split_bf16(x[2] * w, x[3] * w, hi.y, lo.y);
+                *reinterpret_cast<uint2*>(vh + j * ldv + v) = hi;
+                *reinterpret_cast<uint2*>(vl + j * ldv + v) = lo;
             }
         }
-        const bool pairs = (sh.V & 1) == 0;
+        __syncthreads();
+        float* out = U + ((size_t)chunk * sh.H + h) * sh.per;
+        if (sh.normaliser && v0 == 0)
+            for (int d = threadIdx.x; d < sh.D; d += 128) {
+                float sum = 0.0f;
+                for (int j = 0; j < n; ++j) sum = fmaf(coef[j], __bfloat162float(ks[j * ldk + d]), sum);
+                out[(size_t)sh.Dp * sh.Vp + d] = sum;
+            }
+        for (int mt = warp; mt < sh.Dp / 16; mt += 4) {
+            float acc[kCols / 8][4];
 #pragma unroll
-        for (int i = 0; i < kCols / 8; ++i) {
-            const int v = v0 + i * 8 + 2 * tq;
+            for (int i = 0; i < kCols / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+            for (int kk = 0; kk < k_steps; ++kk) {
+                uint32_t a[4];
+                ldmatrix_x4_trans(a, smem_u32(ks + (kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * ldk + mt * 16 + ((lane >> 3) & 1) * 8));
+                const int at = (kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ldv + (lane >> 4) * 8;
 #pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                const int d = mt * 16 + g + r * 8;
-                if (d >= sh.D || v >= sh.V) continue;
-                float* at = out + (size_t)d * sh.V + v;
-                if (pairs) *reinterpret_cast<float2*>(at) = make_float2(acc[i][2 * r], acc[i][2 * r + 1]);
-                else {
-                    at[0] = acc[i][2 * r];
-                    if (v + 1 < sh.V) at[1] = acc[i][2 * r + 1];
+                for (int i = 0; i < kCols / 16; ++i) {
+                    if (2 * i < tiles) {
+                        uint32_t bh[4], bl[4];
+                        ldmatrix_x4_trans(bh, smem_u32(vh + at + i * 16));
+                        ldmatrix_x4_trans(bl, smem_u32(vl + at + i * 16));
+                        mma_bf16(acc[2 * i], a, bh[0], bh[1]);
+                        mma_bf16(acc[2 * i + 1], a, bh[2], bh[3]);
+                        mma_bf16(acc[2 * i], a, bl[0], bl[1]);
+                        mma_bf16(acc[2 * i + 1], a, bl[2], bl[3]);
+                    }
+                }
+            }
+            // rows g of neighbouring lanes (g even and odd) change places, so that a lane holds four numbers of the layout
+#pragma unroll
+            for (int i = 0; i < kCols / 8; ++i) {
+                if (i < tiles) {                          // uniform over the block
+                    const bool odd = g & 1;
+                    const float r0 = __shfl_xor_sync(0xffffffffu, odd ? acc[i][0] : acc[i][1], 4);
+                    const float r1 = __shfl_xor_sync(0xffffffffu, odd ? acc[i][2] : acc[i][3], 4);
+                    const float4 four = odd ? make_float4(r0, acc[i][1], r1, acc[i][3]) : make_float4(acc[i][0], r0, acc[i][2], r1);
+                    const int at = 8 * tq + (odd ? 4 : 0) + (g >> 1);
+                    *reinterpret_cast<float4*>(out + ((size_t)(mt * NT + nt0 + i) * 32 + at) * 4) = four;
                 }
             }
         }
     }
 }
 
-// Along a sequence's chunks: U_c is replaced by the state that enters chunk c; the state behind the last chunk is kept.
+// Along a sequence's chunks: U_c is replaced by the state that enters chunk c (each number as two bfloat16, high and low half of its
+// word; the normaliser's stay float32); the state behind the last chunk is kept.
 __global__ void recurrence_fold_kernel(float* __restrict__ U, const float* __restrict__ total, const Step st, const ChunkShape sh) {
     pdl_wait();
     const int e = blockIdx.x * blockDim.x + threadIdx.x, h = blockIdx.y, s = blockIdx.z;
-    const int DV = sh.D * sh.V, own = DV + (sh.normaliser ? sh.D : 0);
-    if (e >= own) return;
+    const int DVp = sh.Dp * sh.Vp, DV = sh.D * sh.V;
+    if (e >= DVp + (sh.normaliser ? sh.D : 0)) return;
     int first = 0;
     for (int i = 0; i < s; ++i) first += (sh.cu_q[i + 1] - sh.cu_q[i] + kChunk - 1) / kChunk;
     const int nc = (sh.cu_q[s + 1] - sh.cu_q[s] + kChunk - 1) / kChunk;
     float* slot = st.state + (size_t)st.state_slots[s] * st.state_stride;
-    float* kept = e < DV ? slot + (size_t)h * DV + e : slot + (size_t)sh.H * DV + (size_t)h * sh.D + (e - DV);
-    float S = *kept;
+    const bool matrix = e < DVp;
+    float* kept = nullptr;
+    if (matrix) {
+        const int j = e & 3, ln = (e >> 2) & 31, tile = e >> 7, NT = sh.Vp >> 3;
+        const int kk = tile / NT, d = kk * 16 + ((ln & 3) << 1) + (j & 1) + ((j & 2) << 2), v = (tile - kk * NT) * 8 + (ln >> 2);
+        if (d < sh.D && v < sh.V) kept = slot + (size_t)h * DV + (size_t)d * sh.V + v;
+    } else {
+        kept = slot + (size_t)sh.H * DV + (size_t)h * sh.D + (e - DVp);
+    }
+    float S = kept != nullptr ? *kept : 0.0f;
     float* u0 = U + ((size_t)first * sh.H + h) * sh.per + e;
     const float* tot = total + (size_t)first * sh.H + h;
     const size_t step = (size_t)sh.H * sh.per;
     constexpr int kAhead = 8;                // chunks whose own parts are in flight together: they do not depend on the fold
     for (int c0 = 0; c0 < nc; c0 += kAhead) {
-        float ownp[kAhead], dec[kAhead];
+        float own[kAhead], dec[kAhead];
 #pragma unroll
         for (int k = 0; k < kAhead; ++k) {
-            ownp[k] = c0 + k < nc ? u0[(size_t)(c0 + k) * step] : 0.0f;
+            own[k] = c0 + k < nc ? u0[(size_t)(c0 + k) * step] : 0.0f;
             dec[k] = c0 + k < nc ? tot[(size_t)(c0 + k) * sh.H] : 0.0f;
         }
 #pragma unroll
         for (int k = 0; k < kAhead; ++k) {
             if (c0 + k < nc) {
-                u0[(size_t)(c0 + k) * step] = S;
-                S = fmaf(expf(dec[k]), S, ownp[k]);
+                float w = S;
+                if (matrix) {
+                    const bf16 hi = __float2bfloat16_rn(S), lo = __float2bfloat16_rn(S - __bfloat162float(hi));
+                    w = __uint_as_float((uint32_t)__bfloat16_as_ushort(hi) << 16 | __bfloat16_as_ushort(lo));
+                }
+                u0[(size_t)(c0 + k) * step] = w;
+                S = fmaf(expf(dec[k]), S, own[k]);
             }
         }
     }
-    *kept = S;
+    if (kept != nullptr) *kept = S;
 }
 
-// Four warps, 16 tokens each; kCols columns of the values.
+// Four warps, 16 tokens each; kCols columns of the values.  The scores q . k are computed once for the block's heads.
 template <typename T>
-__global__ void __launch_bounds__(128) recurrence_chunk_out_kernel(const Source<T> in, const float* __restrict__ ld, const float* __restrict__ wt,
-                                                                   const ChunkShape sh, const float* __restrict__ S_in,
-                                                                   const float* __restrict__ d_skip, float* __restrict__ out,
-                                                                   float* __restrict__ den) {
+__global__ void __launch_bounds__(128, 4) recurrence_chunk_out_kernel(const Source<T> in, const float* __restrict__ ld, const float* __restrict__ wt,
+                                                                      const ChunkShape sh, const float* __restrict__ S_in,
+                                                                      const float* __restrict__ d_skip, float* __restrict__ out,
+                                                                      float* __restrict__ den) {
     pdl_wait();
     extern __shared__ __align__(16) unsigned char raw_smem[];
     __shared__ float cum[kChunk], weight[kChunk];
-    const int Dp = (sh.D + 15) & ~15, ldk = Dp + kPad, ldv = kCols + kPad;
+    const int ldk = sh.Dp + kPad, ldv = kCols + kPad;
     bf16* qs = reinterpret_cast<bf16*>(raw_smem);         // [kChunk][ldk]
     bf16* ks = qs + kChunk * ldk;                         // [kChunk][ldk]
     bf16* vs = ks + kChunk * ldk;                         // [kChunk][ldv]
-    bf16* Sh = vs + kChunk * ldv;                         // [Dp][ldv] the entering state, high halves
-    bf16* Sl = Sh + Dp * ldv;                             // low halves
-    const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kCols;
+    const int chunk = blockIdx.x, h0 = blockIdx.y * sh.heads, v0 = blockIdx.z * kCols;
     int s, t0, t1;
     if (!find_chunk(sh.cu_q, sh.n_seqs, chunk, s, t0, t1)) return;
     const int n = t1 - t0, cols = min(sh.V - v0, kCols);
-    cumulative_decays(ld, sh.H, h, t0, n, cum);
-    for (int j = threadIdx.x; j < kChunk; j += blockDim.x) weight[j] = j < n ? wt[(size_t)(t0 + j) * sh.H + h] : 0.0f;
-    const size_t qk_at = (size_t)t0 * in.tok + (size_t)(h / in.share) * sh.D;
-    stage_rows(in.q + qk_at, in.tok, n, sh.D, Dp, qs, ldk);
-    stage_rows(in.k + qk_at, in.tok, n, sh.D, Dp, ks, ldk);
-    stage_rows(in.v + (size_t)t0 * in.tok + (size_t)h * sh.V + v0, in.tok, n, cols, kCols, vs, ldv);
-    const float* Sc = S_in + ((size_t)chunk * sh.H + h) * sh.per;
-    {
-        const bool vec = (sh.V & 3) == 0;                 // sh.per is a multiple of four
-        for (int i = threadIdx.x; i < Dp * (kCols / 4); i += blockDim.x) {
-            const int d = i / (kCols / 4), v = (i - d * (kCols / 4)) << 2;
-            float x[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            if (d < sh.D && v < cols) load4(Sc + (size_t)d * sh.V + v0 + v, vec, cols - v, x);
-            uint2 hi, lo;
-            split_bf16(x[0], x[1], hi.x, lo.x);
-            split_bf16(x[2], x[3], hi.y, lo.y);
-            *reinterpret_cast<uint2*>(Sh + d * ldv + v) = hi;
-            *reinterpret_cast<uint2*>(Sl + d * ldv + v) = lo;
-        }
-    }
+    const int NT = sh.Vp >> 3, nt0 = v0 >> 3, tiles = min(NT - nt0, kCols / 8);
+    const size_t qk_at = (size_t)t0 * in.tok + (size_t)(h0 / in.share) * sh.D;
+    stage_rows(in.q + qk_at, in.tok, n, sh.D, sh.Dp, qs, ldk);
+    stage_rows(in.k + qk_at, in.tok, n, sh.D, sh.Dp, ks, ldk);
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tq = lane & 3;
-    if (warp * 16 >= n) return;
+    const bool active = warp * 16 < n;
     const int i0 = warp * 16 + g, i1 = i0 + 8;
-    const float cum0 = cum[i0], cum1 = cum[i1];
-    const int v_tiles = (cols + 15) >> 4;
     const bf16* q_at = qs + (warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ldk + (lane >> 4) * 8;
-    float acc[kCols / 8][4], sc[kChunk / 8][4];
-#pragma unroll
-    for (int i = 0; i < kCols / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    float sc[kChunk / 8][4];
 #pragma unroll
     for (int i = 0; i < kChunk / 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
-    for (int kk = 0; kk < Dp / 16; ++kk) {
-        uint32_t qa[4];
-        ldmatrix_x4(qa, smem_u32(q_at + kk * 16));
-        const int dr = kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
+    if (active) {
+        for (int kk = 0; kk < sh.Dp / 16; ++kk) {
+            uint32_t qa[4];
+            ldmatrix_x4(qa, smem_u32(q_at + kk * 16));
 #pragma unroll
-        for (int i = 0; i < kCols / 16; ++i) {
-            if (i < v_tiles) {
-                uint32_t bh[4], bl[4];
-                ldmatrix_x4_trans(bh, smem_u32(Sh + dr * ldv + i * 16 + (lane >> 4) * 8));
-                ldmatrix_x4_trans(bl, smem_u32(Sl + dr * ldv + i * 16 + (lane >> 4) * 8));
-                mma_bf16(acc[2 * i], qa, bh[0], bh[1]);
-                mma_bf16(acc[2 * i + 1], qa, bh[2], bh[3]);
-                mma_bf16(acc[2 * i], qa, bl[0], bl[1]);
-                mma_bf16(acc[2 * i + 1], qa, bl[2], bl[3]);
+            for (int nn = 0; nn < kChunk / 16; ++nn) {
+                if (nn <= warp) {                         // keys behind the warp's last token are not seen
+                    uint32_t kb[4];
+                    ldmatrix_x4(kb, smem_u32(ks + (nn * 16 + (lane & 7) + ((lane >> 4) << 3)) * ldk + kk * 16 + ((lane >> 3) & 1) * 8));
+                    mma_bf16(sc[2 * nn], qa, kb[0], kb[1]);
+                    mma_bf16(sc[2 * nn + 1], qa, kb[2], kb[3]);
+                }
             }
         }
+#pragma unroll
+        for (int i = 0; i < kChunk / 8; ++i) { sc[i][0] *= sh.q_scale; sc[i][1] *= sh.q_scale; sc[i][2] *= sh.q_scale; sc[i][3] *= sh.q_scale; }
+    }
+    for (int h = h0; h < h0 + sh.heads; ++h) {
+        if (h > h0) __syncthreads();                      // the head before has been read
+        if (warp == 0) chunk_decays<false>(ld, wt, sh.H, h, t0, n, cum, weight);
+        stage_rows(in.v + (size_t)t0 * in.tok + (size_t)h * sh.V + v0, in.tok, n, cols, kCols, vs, ldv);
+        const float* Sc = S_in + ((size_t)chunk * sh.H + h) * sh.per;
+        float acc[kCols / 8][4];
+#pragma unroll
+        for (int i = 0; i < kCols / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+        if (active) {
+            // the entering state comes from memory in the operand's order: 16 bytes a lane and tile, high and low halves in a word
+            const uint4* Sw = reinterpret_cast<const uint4*>(Sc) + (size_t)nt0 * 32 + lane;
+            for (int kk = 0; kk < sh.Dp / 16; ++kk) {
+                uint4 b[kCols / 8];
+#pragma unroll
+                for (int i = 0; i < kCols / 8; ++i) b[i] = i < tiles ? Sw[((size_t)kk * NT + i) * 32] : make_uint4(0, 0, 0, 0);
+                uint32_t qa[4];
+                ldmatrix_x4(qa, smem_u32(q_at + kk * 16));
+#pragma unroll
+                for (int i = 0; i < kCols / 8; ++i)
+                    if (i < tiles) mma_bf16(acc[i], qa, __byte_perm(b[i].x, b[i].y, 0x7632), __byte_perm(b[i].z, b[i].w, 0x7632));
+#pragma unroll
+                for (int i = 0; i < kCols / 8; ++i)
+                    if (i < tiles) mma_bf16(acc[i], qa, __byte_perm(b[i].x, b[i].y, 0x5410), __byte_perm(b[i].z, b[i].w, 0x5410));
+            }
+        }
+        __syncthreads();                                  // the head's decays and values are in shared memory
+        if (!active) continue;
+        const float cum0 = cum[i0], cum1 = cum[i1];
+        const float carry0 = expf(cum0) * sh.q_scale, carry1 = expf(cum1) * sh.q_scale;
+#pragma unroll
+        for (int i = 0; i < kCols / 8; ++i) { acc[i][0] *= carry0; acc[i][1] *= carry0; acc[i][2] *= carry1; acc[i][3] *= carry1; }
+        float size[2] = {0.0f, 0.0f};
 #pragma unroll
         for (int nn = 0; nn < kChunk / 16; ++nn) {
-            if (nn <= warp) {                             // keys behind the warp's last token are not seen
-                uint32_t kb[4];
-                ldmatrix_x4(kb, smem_u32(ks + (nn * 16 + (lane & 7) + ((lane >> 4) << 3)) * ldk + kk * 16 + ((lane >> 3) & 1) * 8));
-                mma_bf16(sc[2 * nn], qa, kb[0], kb[1]);
-                mma_bf16(sc[2 * nn + 1], qa, kb[2], kb[3]);
+            if (nn > warp) continue;
+            float p[2][4];
+#pragma unroll
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int j = nn * 16 + x * 8 + 2 * tq + (e & 1), i = (e >> 1) ? i1 : i0;
+                    const float d = (e >> 1) ? cum1 - cum[j] : cum0 - cum[j];
+                    p[x][e] = (nn < warp || j <= i) ? sc[2 * nn + x][e] * (__expf(d) * weight[j]) : 0.0f;
+                    size[e >> 1] += p[x][e];
+                }
+            uint32_t ph[4], pl[4];
+            split_bf16(p[0][0], p[0][1], ph[0], pl[0]);
+            split_bf16(p[0][2], p[0][3], ph[1], pl[1]);
+            split_bf16(p[1][0], p[1][1], ph[2], pl[2]);
+            split_bf16(p[1][2], p[1][3], ph[3], pl[3]);
+            const int vr = nn * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
+#pragma unroll
+            for (int i = 0; i < kCols / 16; ++i) {
+                if (2 * i < tiles) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, smem_u32(vs + vr * ldv + i * 16 + (lane >> 4) * 8));
+                    mma_bf16(acc[2 * i], ph, b[0], b[1]);
+                    mma_bf16(acc[2 * i + 1], ph, b[2], b[3]);
+                    mma_bf16(acc[2 * i], pl, b[0], b[1]);
+                    mma_bf16(acc[2 * i + 1], pl, b[2], b[3]);
+                }
             }
         }
-    }
-    const float carry0 = expf(cum0) * sh.q_scale, carry1 = expf(cum1) * sh.q_scale;
-#pragma unroll
-    for (int i = 0; i < kCols / 8; ++i) { acc[i][0] *= carry0; acc[i][1] *= carry0; acc[i][2] *= carry1; acc[i][3] *= carry1; }
-    float size[2] = {0.0f, 0.0f};
-#pragma unroll
-    for (int nn = 0; nn < kChunk / 16; ++nn) {
-        if (nn > warp) continue;
-        float p[2][4];
-#pragma unroll
-        for (int x = 0; x < 2; ++x)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int j = nn * 16 + x * 8 + 2 * tq + (e & 1), i = (e >> 1) ? i1 : i0;
-                const float d = (e >> 1) ? cum1 - cum[j] : cum0 - cum[j];
-                p[x][e] = j <= i ? sc[2 * nn + x][e] * sh.q_scale * (__expf(d) * weight[j]) : 0.0f;
-                size[e >> 1] += p[x][e];
+        if (sh.normaliser && v0 == 0) {
+            const float* n_in = Sc + (size_t)sh.Dp * sh.Vp;
+            float part[2] = {0.0f, 0.0f};
+            for (int d = tq; d < sh.D; d += 4) {
+                const float x = n_in[d];
+                part[0] = fmaf(__bfloat162float(qs[i0 * ldk + d]), x, part[0]);
+                part[1] = fmaf(__bfloat162float(qs[i1 * ldk + d]), x, part[1]);
             }
-        uint32_t ph[4], pl[4];
-        split_bf16(p[0][0], p[0][1], ph[0], pl[0]);
-        split_bf16(p[0][2], p[0][3], ph[1], pl[1]);
-        split_bf16(p[1][0], p[1][1], ph[2], pl[2]);
-        split_bf16(p[1][2], p[1][3], ph[3], pl[3]);
-        const int vr = nn * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
+            size[0] = fmaf(carry0, part[0], size[0]);
+            size[1] = fmaf(carry1, part[1], size[1]);
 #pragma unroll
-        for (int i = 0; i < kCols / 16; ++i) {
-            if (i < v_tiles) {
-                uint32_t b[4];
-                ldmatrix_x4_trans(b, smem_u32(vs + vr * ldv + i * 16 + (lane >> 4) * 8));
-                mma_bf16(acc[2 * i], ph, b[0], b[1]);
-                mma_bf16(acc[2 * i + 1], ph, b[2], b[3]);
-                mma_bf16(acc[2 * i], pl, b[0], b[1]);
-                mma_bf16(acc[2 * i + 1], pl, b[2], b[3]);
+            for (int r = 0; r < 2; ++r) {
+                size[r] += __shfl_xor_sync(0xffffffffu, size[r], 1);
+                size[r] += __shfl_xor_sync(0xffffffffu, size[r], 2);
+            }
+            if (tq == 0) {
+                if (i0 < n) den[(size_t)(t0 + i0) * sh.H + h] = size[0];
+                if (i1 < n) den[(size_t)(t0 + i1) * sh.H + h] = size[1];
             }
         }
-    }
-    if (sh.normaliser && v0 == 0) {
-        const float* n_in = Sc + (size_t)sh.D * sh.V;
-        float part[2] = {0.0f, 0.0f};
-        for (int d = tq; d < sh.D; d += 4) {
-            const float x = n_in[d];
-            part[0] = fmaf(__bfloat162float(qs[i0 * ldk + d]), x, part[0]);
-            part[1] = fmaf(__bfloat162float(qs[i1 * ldk + d]), x, part[1]);
-        }
-        size[0] = fmaf(carry0, part[0], size[0]);
-        size[1] = fmaf(carry1, part[1], size[1]);
+        const float skip = d_skip ? d_skip[h] : 0.0f;
+        const bool pairs = (sh.V & 1) == 0, full = n == kChunk && cols == kCols && pairs;
+        float* first = out + ((size_t)(t0 + i0) * sh.H + h) * sh.V + v0 + 2 * tq;
+        const size_t eight_rows = (size_t)8 * sh.H * sh.V;
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            size[r] += __shfl_xor_sync(0xffffffffu, size[r], 1);
-            size[r] += __shfl_xor_sync(0xffffffffu, size[r], 2);
-        }
-        if (tq == 0) {
-            if (i0 < n) den[(size_t)(t0 + i0) * sh.H + h] = size[0];
-            if (i1 < n) den[(size_t)(t0 + i1) * sh.H + h] = size[1];
-        }
-    }
-    const float skip = d_skip ? d_skip[h] : 0.0f;
-    const bool pairs = (sh.V & 1) == 0;
+        for (int i = 0; i < kCols / 8; ++i) {
+            const int v = i * 8 + 2 * tq;
 #pragma unroll
-    for (int i = 0; i < kCols / 8; ++i) {
-        const int v = i * 8 + 2 * tq;
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const int row = r ? i1 : i0;
-            if (row >= n || v >= cols) continue;
-            float x0 = acc[i][2 * r], x1 = acc[i][2 * r + 1];
-            if (d_skip != nullptr) {
-                x0 = fmaf(skip, __bfloat162float(vs[row * ldv + v]), x0);
-                x1 = fmaf(skip, __bfloat162float(vs[row * ldv + v + 1]), x1);
-            }
-            float* at = out + ((size_t)(t0 + row) * sh.H + h) * sh.V + v0 + v;
-            if (pairs) *reinterpret_cast<float2*>(at) = make_float2(x0, x1);
-            else {
-                at[0] = x0;
-                if (v + 1 < cols) at[1] = x1;
+            for (int r = 0; r < 2; ++r) {
+                const int row = r ? i1 : i0;
+                if (!full && (row >= n || v >= cols)) continue;
+                float x0 = acc[i][2 * r], x1 = acc[i][2 * r + 1];
+                if (d_skip != nullptr) {
+                    x0 = fmaf(skip, __bfloat162float(vs[row * ldv + v]), x0);
+                    x1 = fmaf(skip, __bfloat162float(vs[row * ldv + v + 1]), x1);
+                }
+                float* at = first + r * eight_rows + i * 8;
+                if (pairs) *reinterpret_cast<float2*>(at) = make_float2(x0, x1);
+                else {
+                    at[0] = x0;
+                    if (v + 1 < cols) at[1] = x1;
+                }
             }
         }
     }
@@ -825,33 +907,41 @@ int launch_step(StepArgs a, void* y, int tile, cudaStream_t stream) {
 
 size_t smem_state(int D) {
     const size_t Dp = (D + 15) & ~15;
-    return 2 * ((size_t)2 * kChunk * (Dp + kPad) + (size_t)kChunk * (kCols + kPad));
+    return 2 * ((size_t)kChunk * (Dp + kPad) + (size_t)2 * kChunk * (kCols + kPad));
 }
 size_t smem_out(int D) {
     const size_t Dp = (D + 15) & ~15;
-    return 2 * ((size_t)2 * kChunk * (Dp + kPad) + (size_t)kChunk * (kCols + kPad) + 2 * Dp * (kCols + kPad));
+    return 2 * ((size_t)2 * kChunk * (Dp + kPad) + (size_t)kChunk * (kCols + kPad));
 }
 bool chunks_fit(int D) { return smem_out(D) <= 200 * 1024 && smem_state(D) <= 200 * 1024; }
 
+long chunk_words(int D, int V, int normaliser) {
+    return ((long)((D + 15) & ~15) * ((V + 7) & ~7) + (normaliser ? D : 0) + 3) / 4 * 4;
+}
+
 template <typename T>
-int launch_chunks(const Source<T>& in, const float* ld, const float* wt, const ChunkShape& sh, const Step& st, float* U, float* total,
+int launch_chunks(const Source<T>& in, const float* ld, const float* wt, ChunkShape sh, const Step& st, float* U, float* total,
                   int max_chunks, const float* d_skip, float* raw, float* den, cudaStream_t stream) {
     const int tiles = (sh.V + kCols - 1) / kCols;
     if (tiles > 65535 || sh.H > 65535 || st.n_seqs > 65535) return PB_ERR_TOO_LARGE;
+    sh.Dp = (sh.D + 15) & ~15;
+    sh.Vp = (sh.V + 7) & ~7;
+    sh.per = chunk_words(sh.D, sh.V, sh.normaliser);
+    // neighbouring heads that read the same q and k share a block (their keys are staged and their scores computed once), as long
+    // as there are blocks for every SM
+    sh.heads = 1;
+    while (sh.heads < 4 && in.share % (2 * sh.heads) == 0 && (long)max_chunks * tiles * sh.H / (2 * sh.heads) >= 2 * 148) sh.heads *= 2;
     int rc = allow_smem(recurrence_chunk_state_kernel<T>, smem_state(sh.D));
     if (rc == 0) rc = allow_smem(recurrence_chunk_out_kernel<T>, smem_out(sh.D));
     if (rc != 0) return rc;
-    rc = launch_pdl(recurrence_chunk_state_kernel<T>, dim3(max_chunks, sh.H, tiles), dim3(128), smem_state(sh.D), stream, in, ld, wt, sh, U,
-                    total);
+    const dim3 grid(max_chunks, sh.H / sh.heads, tiles);
+    rc = launch_pdl(recurrence_chunk_state_kernel<T>, grid, dim3(128), smem_state(sh.D), stream, in, ld, wt, sh, U, total);
     if (rc != 0) return rc;
-    const int own = sh.D * sh.V + (sh.normaliser ? sh.D : 0);
+    const int own = sh.Dp * sh.Vp + (sh.normaliser ? sh.D : 0);
     rc = launch_pdl(recurrence_fold_kernel, dim3((own + 255) / 256, sh.H, st.n_seqs), dim3(256), 0, stream, U, (const float*)total, st, sh);
     if (rc != 0) return rc;
-    return launch_pdl(recurrence_chunk_out_kernel<T>, dim3(max_chunks, sh.H, tiles), dim3(128), smem_out(sh.D), stream, in, ld, wt, sh,
-                      (const float*)U, d_skip, raw, den);
+    return launch_pdl(recurrence_chunk_out_kernel<T>, grid, dim3(128), smem_out(sh.D), stream, in, ld, wt, sh, (const float*)U, d_skip, raw, den);
 }
-
-long chunk_floats(int D, int V, int normaliser) { return ((long)D * V + (normaliser ? D : 0) + 3) / 4 * 4; }
 
 }  // namespace
 
@@ -868,7 +958,7 @@ PB_EXPORT int pb_recurrence_supported(int D, int V) {
 // chunks' totals [max_chunks, H] and their states.
 PB_EXPORT long pb_recurrence_workspace(int n, int H, int D, int V, int max_chunks, int normaliser) {
     const long raw = ((long)n * H * V + 3) / 4 * 4, scalars = ((long)4 * n * H + 3) / 4 * 4, totals = ((long)max_chunks * H + 3) / 4 * 4;
-    return raw + scalars + totals + (long)max_chunks * H * chunk_floats(D, V, normaliser);
+    return raw + scalars + totals + (long)max_chunks * H * chunk_words(D, V, normaliser);
 }
 
 // rows float32 [n, stride]: q (H*D) | k (H*D) | v (H*V) | g (H*V) | i (H) | f (H); biases float32 [H]; norm_w float32 [H*V]; state:
@@ -909,14 +999,14 @@ PB_EXPORT int pb_matrix_memory(int dtype, const float* rows, long stride, const 
     float *wt = ld + (long)n * H, *floor = wt + (long)n * H, *den = floor + (long)n * H;
     float* total = ld + ((long)4 * n * H + 3) / 4 * 4;
     float* U = total + ((long)(max_chunks > 0 ? max_chunks : 0) * H + 3) / 4 * 4;
-    const int threads = n >= 256 * n_seqs ? 512 : 128;
+    const int threads = n >= 512 * n_seqs ? 1024 : n >= 128 * n_seqs ? 512 : 128;
     int rc = launch_pdl(memory_gates_kernel, dim3(H, n_seqs), dim3(threads), 0, stream, rows, stride, a.i_off, a.f_off, i_bias, f_bias, cap, st,
                         HDV + (long)H * D, H, ld, wt, floor);
     if (rc != 0) return rc;
     if (max_chunks > 0) {
         if (dtype != PB_BF16 || !chunks_fit(D)) return PB_ERR_TOO_LARGE;
         const Source<float> in{rows, rows + a.k_off, rows + a.v_off, stride, 1};
-        const ChunkShape sh{cu_q, n_seqs, H, D, V, 1, chunk_floats(D, V, 1), q_scale};
+        const ChunkShape sh{cu_q, n_seqs, H, D, V, 1, 0, 0, 0, q_scale, 1};
         rc = launch_chunks<float>(in, ld, wt, sh, st, U, total, max_chunks, nullptr, raw, den, stream);
     } else {
         const int tile = step_tile(D, V + 1, 128);
@@ -972,7 +1062,7 @@ PB_EXPORT int pb_state_space(int dtype, const float* rows, long stride, const fl
         if (rc != 0) return rc;
         const bf16* x = (const bf16*)xbc;
         const Source<bf16> in{x + inner + G * D, x + inner, x, channels, H / G};
-        const ChunkShape sh{cu_q, n_seqs, H, D, V, 0, chunk_floats(D, V, 0), 1.0f};
+        const ChunkShape sh{cu_q, n_seqs, H, D, V, 0, 0, 0, 0, 1.0f, 1};
         rc = launch_chunks<bf16>(in, ld, wt, sh, st, U, total, max_chunks, d_skip, raw, nullptr, stream);
     } else {
         StepArgs a{};

@@ -31,26 +31,57 @@ using namespace pb;
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 
-template <typename TIn, typename T>
+constexpr int kConvRun = 16;         // tokens a thread walks
+
+// The convolution at token t (index i of its portion) of channel c.
+template <typename TIn>
+__device__ __forceinline__ float conv_at(const TIn* __restrict__ in, long in_tok, const float* __restrict__ taps, float bias,
+                                         const float* __restrict__ tail, int t, int i, int c, int n_taps) {
+    float acc = bias;
+    for (int tau = 0; tau < n_taps; ++tau) {
+        const int back = n_taps - 1 - tau;
+        const float v = (i - back >= 0) ? to_float(in[(size_t)(t - back) * in_tok + c]) : tail[(size_t)c * (n_taps - 1) + n_taps - 1 + i - back];
+        acc = fmaf(taps[(size_t)c * n_taps + tau], v, acc);
+    }
+    return acc;
+}
+
+// A thread takes one channel of `run` neighbouring tokens.  Where those are kConvRun tokens in the midst of one portion and the
+// taps are kTaps, it reads each input once and keeps the taps in registers (the same sums in the same order).
+template <typename TIn, typename T, int kTaps>
 __global__ void __launch_bounds__(256)
 causal_conv_silu_kernel(const TIn* __restrict__ in, long in_tok, const float* __restrict__ taps, const float* __restrict__ bias,
                         const float* __restrict__ arena, long slot_stride, long tail_offset, const int* __restrict__ cu_q,
                         const int* __restrict__ seq_of_token, const int* __restrict__ state_slots, T* __restrict__ out,
-                        int channels, int n_taps) {
+                        int channels, int n_taps, int n_tokens, int run) {
     pdl_wait();         // may have come onto the SMs while the product before it was ending: nothing is touched before that one is done
-    const int t = blockIdx.x;
+    const int t0 = blockIdx.x * run, t1 = min(t0 + run, n_tokens);
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= channels) return;
-    const int s = seq_of_token[t];
-    const int i = t - cu_q[s];                          // index within the portion
-    const float* tail = arena + (size_t)state_slots[s] * slot_stride + tail_offset + (size_t)c * (n_taps - 1);
-    float acc = bias[c];
-    for (int tau = 0; tau < n_taps; ++tau) {
-        const int back = n_taps - 1 - tau;
-        const float v = (i - back >= 0) ? to_float(in[(size_t)(t - back) * in_tok + c]) : tail[n_taps - 1 + i - back];
-        acc = fmaf(taps[(size_t)c * n_taps + tau], v, acc);
+    const float b = bias[c];
+    if (kTaps > 0 && t1 - t0 == kConvRun) {
+        const int s = seq_of_token[t0];
+        if (s == seq_of_token[t1 - 1] && t0 - cu_q[s] >= kTaps - 1) {        // uniform over the block
+            float w[kTaps > 0 ? kTaps : 1], x[kConvRun + kTaps];
+#pragma unroll
+            for (int k = 0; k < kTaps; ++k) w[k] = taps[(size_t)c * kTaps + k];
+#pragma unroll
+            for (int k = 0; k < kConvRun + kTaps - 1; ++k) x[k] = to_float(in[(size_t)(t0 - (kTaps - 1) + k) * in_tok + c]);
+#pragma unroll
+            for (int k = 0; k < kConvRun; ++k) {
+                float acc = b;
+#pragma unroll
+                for (int tau = 0; tau < kTaps; ++tau) acc = fmaf(w[tau], x[k + tau], acc);
+                out[(size_t)(t0 + k) * channels + c] = from_float<T>(silu_f(acc));
+            }
+            return;
+        }
     }
-    out[(size_t)t * channels + c] = from_float<T>(silu_f(acc));
+    for (int t = t0; t < t1; ++t) {
+        const int s = seq_of_token[t];
+        const float* tail = arena + (size_t)state_slots[s] * slot_stride + tail_offset;
+        out[(size_t)t * channels + c] = from_float<T>(silu_f(conv_at(in, in_tok, taps, b, tail, t, t - cu_q[s], c, n_taps)));
+    }
 }
 
 constexpr int kStage = 16;          // tokens staged per round
@@ -477,14 +508,23 @@ PB_EXPORT int pb_causal_conv_silu(int in_dtype, int dtype, const void* in, long 
                                   const int* state_slots, void* out, int n_tokens, int channels, int n_taps, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (channels <= 0 || n_taps < 1) return PB_ERR_BAD_SIZE;
-    dim3 grid(n_tokens, (channels + 255) / 256);
+    const int run = n_tokens >= 8 * kConvRun ? kConvRun : 1;       // a few tokens: each in a block of its own
+    dim3 grid((n_tokens + run - 1) / run, (channels + 255) / 256);
     if (grid.y > 65535) return PB_ERR_TOO_LARGE;
-#define PB_CONV(TI, T) return launch_pdl(causal_conv_silu_kernel<TI, T>, grid, dim3(256), 0, stream, (const TI*)in, in_tok, taps, bias, arena, \
-                                         slot_stride, tail_offset, cu_q, seq_of_token, state_slots, (T*)out, channels, n_taps)
+#define PB_CONV_TAPS(TI, T, K) return launch_pdl(causal_conv_silu_kernel<TI, T, K>, grid, dim3(256), 0, stream, (const TI*)in, in_tok, taps, bias, arena, \
+                                                 slot_stride, tail_offset, cu_q, seq_of_token, state_slots, (T*)out, channels, n_taps, n_tokens, run)
+#define PB_CONV(TI, T)                                  \
+    do {                                                \
+        if (n_taps == 4) PB_CONV_TAPS(TI, T, 4);        \
+        if (n_taps == 3) PB_CONV_TAPS(TI, T, 3);        \
+        if (n_taps == 2) PB_CONV_TAPS(TI, T, 2);        \
+        PB_CONV_TAPS(TI, T, 0);                         \
+    } while (0)
     if (in_dtype == PB_F32 && dtype == PB_F32) PB_CONV(float, float);
     if (in_dtype == PB_BF16 && dtype == PB_BF16) PB_CONV(__nv_bfloat16, __nv_bfloat16);
     if (in_dtype == PB_F32 && dtype == PB_BF16) PB_CONV(float, __nv_bfloat16);
 #undef PB_CONV
+#undef PB_CONV_TAPS
     return PB_ERR_BAD_DTYPE;
 }
 
