@@ -92,20 +92,21 @@ __device__ __forceinline__ bool slot_ok(int slot, int page_size, const PoolBound
 // The gating of a fused gate/up product, carried with the product's `inter` (the output's width) so that it reaches every
 // epilogue: out = g' * sigmoid(alpha * g') * (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).  SwiGLU is
 // limit = inf, alpha = 1, shift = 0 (the formula then is silu(g) * u to the last bit); a clamped gated unit gives its own.
-// alpha = inf is the sigmoid's limit, a step at zero: g' * [g' > 0] = max(g', 0), the ReLU-gated unit.
+// alpha = inf is the sigmoid's limit, a step at zero: g' * [g' > 0] = max(g', 0), the ReLU-gated unit.  It is held as the largest
+// finite number, with which the formula gives just that (exp of an overflowed product is 0 or inf; zero stays zero) and the
+// epilogues need no branch.
 // The host sets what the next gated launches use (pb_set_gating) and the launchers read it with gating_now(inter).
 struct GatedInter {
     int n;
     float limit, alpha, shift;
     __host__ __device__ GatedInter(int n_ = 0, float limit_ = __builtin_huge_valf(), float alpha_ = 1.0f, float shift_ = 0.0f)
-        : n(n_), limit(limit_), alpha(alpha_), shift(shift_) {}
+        : n(n_), limit(limit_), alpha(alpha_ > 3.402823466e38f ? 3.402823466e38f : alpha_), shift(shift_) {}
     __host__ __device__ operator int() const { return n; }
 };
 GatedInter gating_now(int inter);        // host side: `inter` with the gating that pb_set_gating set last
 __device__ __forceinline__ float gated(float g, float u, const GatedInter& p) {
     g = fminf(g, p.limit);
     u = fminf(fmaxf(u, -p.limit), p.limit);
-    if (p.alpha == __builtin_huge_valf()) return fmaxf(g, 0.0f) * (u + p.shift);          // uniform over the grid
     return g / (1.0f + expf(-p.alpha * g)) * (u + p.shift);
 }
 
